@@ -64,6 +64,15 @@ __device__ __forceinline__ float mv_block_sum(float v, float* scratch) {
     return scratch[32];
 }
 
+// The gated activations of a feed-forward: silu(g) * u, and g' * sigmoid(alpha g') * (u' + 1) with
+// g' = min(g, limit), u' = u cut off at -limit and limit.
+__device__ __forceinline__ float mv_glu_silu(float g, float u) { return g / (1.0f + expf(-g)) * u; }
+__device__ __forceinline__ float mv_glu_clamped(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+
 // Loads 8 consecutive elements (16-byte aligned for bf16, 32-byte span for
 // f32) into floats.
 __device__ __forceinline__ void mv_load8(const float* p, float* out) {

@@ -304,13 +304,14 @@ MV_API int mv_delay(long long us, cudaStream_t stream) {
 // x = table[token] + bigram[r], r = (previous token * mul_prev + token * mul_cur) mod buckets, or row `buckets`
 // (the table's last) for the token at position 0.  The previous token of a step's first token is what the
 // sequence kept (prev[slot]); the block of a sequence's first row in the step also writes the sequence's last
-// token of the step there, after it has read the old one.  ``kept`` (or null) gets a second copy of the rows.
-template <typename T>
+// token of the step there, after it has read the old one.  ``kept`` (or null) gets a second copy of the rows,
+// ``rounded`` (or null) the rows in the model's dtype.
+template <typename T, typename TO>
 __global__ void embed_bigram_kernel(const T* __restrict__ table, const T* __restrict__ bigram, const int* __restrict__ tok,
                                     const int* __restrict__ positions, const int* __restrict__ seq_of,
                                     const int* __restrict__ cu, const int* __restrict__ slots, int* __restrict__ prev,
-                                    float* __restrict__ x, float* __restrict__ kept, int H, int buckets,
-                                    long long mul_prev, long long mul_cur) {
+                                    float* __restrict__ x, float* __restrict__ kept, TO* __restrict__ rounded, int H,
+                                    int buckets, long long mul_prev, long long mul_cur) {
     mv_pdl_begin();
     __shared__ int row_s;
     const int n = blockIdx.x;
@@ -336,23 +337,28 @@ __global__ void embed_bigram_kernel(const T* __restrict__ table, const T* __rest
         const float v = mv_to_f32(row[h]) + mv_to_f32(brow[h]);
         x[(size_t)n * H + h] = v;
         if (kept) kept[(size_t)n * H + h] = v;
+        if (rounded) rounded[(size_t)n * H + h] = mv_from_f32<TO>(v);
     }
 }
 
 MV_GUARD_SETTER(elementwise)
 
 MV_API int mv_embed_bigram(const void* table, const void* bigram, int table_dtype, const int* tok, const int* positions,
-                           const int* seq_of, const int* cu, const int* slots, int* prev, float* x, float* kept, int N,
-                           int H, int buckets, long long mul_prev, long long mul_cur, cudaStream_t stream) {
+                           const int* seq_of, const int* cu, const int* slots, int* prev, float* x, float* kept,
+                           void* rounded, int rounded_dtype, int N, int H, int buckets, long long mul_prev,
+                           long long mul_cur, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (buckets < 1) return (int)cudaErrorInvalidValue;
     const int threads = H >= 1024 ? 256 : 128;
-    if (table_dtype == MV_DT_BF16)
-        mv_launch(embed_bigram_kernel<__nv_bfloat16>, N, threads, 0, stream, (const __nv_bfloat16*)table,
-                  (const __nv_bfloat16*)bigram, tok, positions, seq_of, cu, slots, prev, x, kept, H, buckets, mul_prev, mul_cur);
-    else
-        mv_launch(embed_bigram_kernel<float>, N, threads, 0, stream, (const float*)table, (const float*)bigram, tok,
-                  positions, seq_of, cu, slots, prev, x, kept, H, buckets, mul_prev, mul_cur);
+#define EB_LAUNCH(T, TO)                                                                                              \
+    mv_launch(embed_bigram_kernel<T, TO>, N, threads, 0, stream, (const T*)table, (const T*)bigram, tok, positions, seq_of, \
+              cu, slots, prev, x, kept, (TO*)rounded, H, buckets, mul_prev, mul_cur)
+    if (table_dtype == MV_DT_BF16) {
+        if (rounded && rounded_dtype == MV_DT_F32) EB_LAUNCH(__nv_bfloat16, float); else EB_LAUNCH(__nv_bfloat16, __nv_bfloat16);
+    } else {
+        if (rounded && rounded_dtype == MV_DT_BF16) EB_LAUNCH(float, __nv_bfloat16); else EB_LAUNCH(float, float);
+    }
+#undef EB_LAUNCH
     return mv_launch_status();
 }
 

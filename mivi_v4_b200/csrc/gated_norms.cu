@@ -378,63 +378,168 @@ MV_API int mv_rmsnorm_add_layernorm(const float* y, const float* w, float eps, f
     return mv_launch_status();
 }
 
+// ------------------------- a norm after the sum, with a gate on the sublayer's result
+// x <- alpha x + sigmoid(z + b) * (s1 y1 + s2 y2) element by element (z null: no gate; b null: no bias; y2 null: s1 y1),
+// then resid[n, :] = x / sqrt(mean(x^2) + eps) * w: a layer whose norm sits behind the residual sum, so that the stream
+// itself is normed.  ``rounded`` (or null) gets the completed row in the model's dtype, for the sublayer that reads it
+// next.  z has a row stride of its own (the gate's logits may be columns of a wider product).
+__device__ __forceinline__ float sn_join(float x, float alpha, float v, bool gated, float z) {
+    return fmaf(alpha, x, gated ? v / (1.0f + expf(-z)) : v);
+}
+
+template <typename TO>
+__global__ void sum_norm_kernel(const float* __restrict__ y1, float s1, const float* __restrict__ y2, float s2,
+                                const float* __restrict__ z, long long ldz, const float* __restrict__ b,
+                                float* __restrict__ resid, float alpha, const float* __restrict__ w, float eps,
+                                TO* __restrict__ rounded, int H) {
+    mv_pdl_begin();
+    __shared__ float scratch[33];
+    const size_t base = (size_t)blockIdx.x * H;
+    const float* zr = z ? z + (size_t)blockIdx.x * ldz : nullptr;
+    float ss = 0.f;
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {          // a thread reads back only what it wrote itself
+        const float v = y2 ? fmaf(s2, y2[base + h], s1 * y1[base + h]) : s1 * y1[base + h];
+        const float r = sn_join(resid[base + h], alpha, v, zr != nullptr, zr ? zr[h] + (b ? b[h] : 0.f) : 0.f);
+        resid[base + h] = r;
+        ss = fmaf(r, r, ss);
+    }
+    const float scale = 1.0f / sqrtf(mv_block_sum(ss, scratch) / (float)H + eps);
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {
+        const float r = resid[base + h] * scale * w[h];
+        resid[base + h] = r;
+        if (rounded) rounded[base + h] = mv_from_f32<TO>(r);
+    }
+}
+
+// The same with four values a load, a row's values kept in registers between the two passes: for rows of a
+// multiple of 4 and at most 8 values a thread, 16-byte aligned.
+template <typename TO>
+__global__ void __launch_bounds__(512)
+sum_norm_vec_kernel(const float* __restrict__ y1, float s1, const float* __restrict__ y2, float s2,
+                    const float* __restrict__ z, long long ldz, const float* __restrict__ b, float* __restrict__ resid,
+                    float alpha, const float* __restrict__ w, float eps, TO* __restrict__ rounded, int H) {
+    mv_pdl_begin();
+    __shared__ float scratch[33];
+    const size_t base = (size_t)blockIdx.x * H;
+    const int H4 = H >> 2;
+    float4 r[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int h4 = threadIdx.x + i * blockDim.x;
+        r[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (h4 < H4) {
+            const float4 a = reinterpret_cast<const float4*>(y1 + base)[h4];
+            float4 v = make_float4(s1 * a.x, s1 * a.y, s1 * a.z, s1 * a.w);
+            if (y2) {
+                const float4 c = reinterpret_cast<const float4*>(y2 + base)[h4];
+                v = make_float4(fmaf(s2, c.x, v.x), fmaf(s2, c.y, v.y), fmaf(s2, c.z, v.z), fmaf(s2, c.w, v.w));
+            }
+            const float4 x = reinterpret_cast<const float4*>(resid + base)[h4];
+            float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (z) {
+                g = reinterpret_cast<const float4*>(z + (size_t)blockIdx.x * ldz)[h4];
+                if (b) {
+                    const float4 bb = reinterpret_cast<const float4*>(b)[h4];
+                    g = make_float4(g.x + bb.x, g.y + bb.y, g.z + bb.z, g.w + bb.w);
+                }
+            }
+            const bool gated = z != nullptr;
+            r[i] = make_float4(sn_join(x.x, alpha, v.x, gated, g.x), sn_join(x.y, alpha, v.y, gated, g.y),
+                               sn_join(x.z, alpha, v.z, gated, g.z), sn_join(x.w, alpha, v.w, gated, g.w));
+            ss = fmaf(r[i].x, r[i].x, ss); ss = fmaf(r[i].y, r[i].y, ss);
+            ss = fmaf(r[i].z, r[i].z, ss); ss = fmaf(r[i].w, r[i].w, ss);
+        }
+    }
+    const float scale = 1.0f / sqrtf(mv_block_sum(ss, scratch) / (float)H + eps);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int h4 = threadIdx.x + i * blockDim.x;
+        if (h4 < H4) {
+            const float4 ww = reinterpret_cast<const float4*>(w)[h4];
+            const float4 o = make_float4(r[i].x * scale * ww.x, r[i].y * scale * ww.y, r[i].z * scale * ww.z, r[i].w * scale * ww.w);
+            reinterpret_cast<float4*>(resid + base)[h4] = o;
+            if (rounded) mv_store4(rounded + base + 4 * (size_t)h4, o.x, o.y, o.z, o.w);
+        }
+    }
+}
+
+MV_API int mv_sum_norm(const float* y1, float s1, const float* y2, float s2, const float* z, long long ldz, const float* b,
+                       float* resid, float alpha, const float* w, float eps, void* rounded, int rounded_dtype, int N, int H,
+                       cudaStream_t stream) {
+    if (N <= 0) return 0;
+    const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
+    const bool aligned = (((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)z | (uintptr_t)b | (uintptr_t)resid | (uintptr_t)w |
+                           (uintptr_t)rounded) & 15) == 0 && (!z || ldz % 4 == 0);
+    const bool narrow = rounded && rounded_dtype == MV_DT_BF16;
+#define SN_LAUNCH(KERNEL, TO) \
+    mv_launch(KERNEL<TO>, N, threads, 0, stream, y1, s1, y2, s2, z, ldz, b, resid, alpha, w, eps, (TO*)rounded, H)
+    if (H % 4 == 0 && H / 4 <= 2 * threads && aligned) {
+        if (narrow) SN_LAUNCH(sum_norm_vec_kernel, __nv_bfloat16); else SN_LAUNCH(sum_norm_vec_kernel, float);
+    } else {
+        if (narrow) SN_LAUNCH(sum_norm_kernel, __nv_bfloat16); else SN_LAUNCH(sum_norm_kernel, float);
+    }
+#undef SN_LAUNCH
+    return mv_launch_status();
+}
+
 // ------------------------------------------------------ clamped gated activation
 // h[n, f] = g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit);
-// gate = gu[n, f], up = gu[n, F + f].
+// gate = gu[n, f], up = gu[n, F + f], or with `group` they alternate in groups of that many columns.
 template <typename TO>
-__global__ void glu_clamped_kernel(const float* __restrict__ gu, TO* __restrict__ h, long long total, int F, float limit,
-                                   float alpha) {
+__global__ void glu_clamped_kernel(const float* __restrict__ gu, TO* __restrict__ h, long long total, int F, int group,
+                                   float limit, float alpha) {
     mv_pdl_begin();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     const long long n = i / F;
     const int f = (int)(i - n * F);
-    const float g = fminf(gu[n * 2 * F + f], limit);
-    const float u = fminf(fmaxf(gu[n * 2 * F + F + f], -limit), limit);
-    h[i] = mv_from_f32<TO>(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
+    const float* row = gu + n * 2 * F;
+    const int gi = group ? (f / group) * 2 * group + f % group : f;
+    h[i] = mv_from_f32<TO>(mv_glu_clamped(row[gi], row[gi + (group ? group : F)], limit, alpha));
 }
 
-// The same with four consecutive features a thread (16-byte loads): F a multiple of 4, 16-byte aligned rows.
+// The same with four consecutive features a thread (16-byte loads): F and `group` multiples of 4, 16-byte aligned rows.
 template <typename TO>
 __global__ void __launch_bounds__(256)
-glu_clamped_vec_kernel(const float* __restrict__ gu, TO* __restrict__ h, long long total4, int F, float limit, float alpha) {
+glu_clamped_vec_kernel(const float* __restrict__ gu, TO* __restrict__ h, long long total4, int F, int group, float limit,
+                       float alpha) {
     mv_pdl_begin();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total4) return;
     const int F4 = F >> 2;
     const long long n = i / F4;
     const int f = (int)(i - n * F4) << 2;
-    const float4 g4 = *reinterpret_cast<const float4*>(gu + n * 2 * F + f);
-    const float4 u4 = *reinterpret_cast<const float4*>(gu + n * 2 * F + F + f);
+    const float* row = gu + n * 2 * F;
+    const int gi = group ? (f / group) * 2 * group + f % group : f;
+    const float4 g4 = *reinterpret_cast<const float4*>(row + gi);
+    const float4 u4 = *reinterpret_cast<const float4*>(row + gi + (group ? group : F));
     const float gs[4] = {g4.x, g4.y, g4.z, g4.w}, us[4] = {u4.x, u4.y, u4.z, u4.w};
     float y[4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-        const float g = fminf(gs[j], limit);
-        const float u = fminf(fmaxf(us[j], -limit), limit);
-        y[j] = g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
-    }
+    for (int j = 0; j < 4; ++j) y[j] = mv_glu_clamped(gs[j], us[j], limit, alpha);
     mv_store4(h + n * F + f, y[0], y[1], y[2], y[3]);
 }
 
-MV_API int mv_glu_clamped(const float* gu, void* h, int h_dtype, int N, int F, float limit, float alpha,
+MV_API int mv_glu_clamped(const float* gu, void* h, int h_dtype, int N, int F, int group, float limit, float alpha,
                           cudaStream_t stream) {
     const long long total = (long long)N * F;
     if (total <= 0) return 0;
-    if (F % 4 == 0 && (((uintptr_t)gu | (uintptr_t)h) & 15) == 0) {
+    if (group < 0 || (group && F % group)) return (int)cudaErrorInvalidValue;
+    if (F % 4 == 0 && group % 4 == 0 && (((uintptr_t)gu | (uintptr_t)h) & 15) == 0) {
         const unsigned blocks4 = (unsigned)((total / 4 + 255) / 256);
         if (h_dtype == MV_DT_BF16)
-            mv_launch(glu_clamped_vec_kernel<__nv_bfloat16>, blocks4, 256, 0, stream, gu, (__nv_bfloat16*)h, total / 4, F, limit,
-                      alpha);
+            mv_launch(glu_clamped_vec_kernel<__nv_bfloat16>, blocks4, 256, 0, stream, gu, (__nv_bfloat16*)h, total / 4, F, group,
+                      limit, alpha);
         else
-            mv_launch(glu_clamped_vec_kernel<float>, blocks4, 256, 0, stream, gu, (float*)h, total / 4, F, limit, alpha);
+            mv_launch(glu_clamped_vec_kernel<float>, blocks4, 256, 0, stream, gu, (float*)h, total / 4, F, group, limit, alpha);
         return mv_launch_status();
     }
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (h_dtype == MV_DT_BF16)
-        mv_launch(glu_clamped_kernel<__nv_bfloat16>, blocks, 256, 0, stream, gu, (__nv_bfloat16*)h, total, F, limit, alpha);
+        mv_launch(glu_clamped_kernel<__nv_bfloat16>, blocks, 256, 0, stream, gu, (__nv_bfloat16*)h, total, F, group, limit, alpha);
     else
-        mv_launch(glu_clamped_kernel<float>, blocks, 256, 0, stream, gu, (float*)h, total, F, limit, alpha);
+        mv_launch(glu_clamped_kernel<float>, blocks, 256, 0, stream, gu, (float*)h, total, F, group, limit, alpha);
     return mv_launch_status();
 }
 

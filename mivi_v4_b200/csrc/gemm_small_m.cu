@@ -430,13 +430,13 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __
             ss = mv_warp_sum(ss);
             v *= 1.0f / sqrtf(ss * link.inv_dim + link.eps);
         }
-        if (bias && r < ROWS && n < N) v += bias[n];
-        if (mode == 3) {
+        if (bias && mode != 4 && r < ROWS && n < N) v += bias[n];
+        if (mode >= 3) {
             // ROWS == 32: lanes 0-15 hold gate rows, lanes 16-31 the up rows of the same features
             const float up = __shfl_down_sync(0xffffffffu, v, 16);
             if (lane < 16 && n + 16 < N)
                 ((__nv_bfloat16*)out)[(size_t)m * ldo + (n >> 5) * 16 + lane] =
-                    __float2bfloat16_rn(v / (1.0f + expf(-v)) * up);
+                    __float2bfloat16_rn(mode == 4 ? mv_glu_clamped(v, up, bias[n], bias[N]) : mv_glu_silu(v, up));
         } else {
             float sq = 0.f;
             if (r < ROWS && n < N) {
@@ -513,10 +513,11 @@ int launch(const void* W, const void* X, const float* bias, void* out, int mode,
 
 // Rows of W per block for this shape: 32 halve the re-reads of X and are what the SwiGLU
 // epilogue needs; 16 keep more blocks for a narrow matrix.  (Also the rows behind one tile sum.)
-MV_API int mv_gemm_small_m_tile_rows(int N, int mode) { return (N >= 32 * 2 * 148 || mode == 3) ? 32 : 16; }
+MV_API int mv_gemm_small_m_tile_rows(int N, int mode) { return (N >= 32 * 2 * 148 || mode >= 3) ? 32 : 16; }
 
 // mode: 0 store float32, 1 store bfloat16, 2 add into float32, 3 SwiGLU (W rows in
-// groups of 16 gate + 16 up; out is bfloat16 [M, N/2] with row stride ldo).  Needs
+// groups of 16 gate + 16 up; out is bfloat16 [M, N/2] with row stride ldo), 4 the clamped gated activation over
+// such rows (bias [N + 1]: a limit a row of W, then alpha).  Needs
 // 1 <= M <= 64, K a multiple of 8, and 16-byte aligned operands.
 // scale_part (or null): [M][scale_stride] of which n_scale_part sums of squares per token; every token's
 // results are multiplied by rsqrt(sum / dim + eps) before bias and activation.  emit_x (or null, mode 2
@@ -529,7 +530,7 @@ MV_API int mv_gemm_small_m(const void* X, const void* W, const float* bias, void
                            int emit_stride, const void* next_w, long long next_bytes, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 64 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode == 3 && N % 32) return (int)cudaErrorInvalidValue;
+    if (mode >= 3 && (N % 32 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
     if (emit_x && (mode != 2 || ldo != N || !emit_g || !emit_part ||
                    emit_stride < (N + mv_gemm_small_m_tile_rows(N, 2) - 1) / mv_gemm_small_m_tile_rows(N, 2)))
         return (int)cudaErrorInvalidValue;

@@ -359,7 +359,7 @@ int launch(const void* X, const void* W, const float* bias, void* out, int mode,
 
 // The grouped form: X [M, K] sorted by group, W [w_rows, w_cols] holding every group's matrix.
 template <int BN, int STAGES>
-int launch_grouped(const void* X, const void* W, void* out, int mode, int M, int N, int K, int ldo, int w_rows, int w_cols,
+int launch_grouped(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo, int w_rows, int w_cols,
                    const int* tile_group, int b_row_step, int b_k_step, int* err, cudaStream_t stream) {
     using L = SmemLayout<BN, STAGES>;
     CUtensorMap ma, mb;
@@ -370,7 +370,7 @@ int launch_grouped(const void* X, const void* W, void* out, int mode, int M, int
         attr_set = true;
     }
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
-    gemm_tc_kernel<BN, STAGES><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, nullptr, out, mode, M, N, K, ldo, RowScale{}, err,
+    gemm_tc_kernel<BN, STAGES><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, RowScale{}, err,
                                                                    tile_group, b_row_step, b_k_step);
     return mv_launch_status();
 }
@@ -378,7 +378,8 @@ int launch_grouped(const void* X, const void* W, void* out, int mode, int M, int
 }  // namespace
 
 // mode: 0 store float32, 1 store bfloat16, 2 add into float32, 3 SwiGLU (W rows in groups
-// of 16 gate + 16 up; out is bfloat16 [M, N/2] with row stride ldo).  ``err`` points to a
+// of 16 gate + 16 up; out is bfloat16 [M, N/2] with row stride ldo), 4 the clamped gated activation over such rows
+// (bias [N + 1]: a limit a row of W, then alpha).  ``err`` points to a
 // device int that a block sets (1 producer, 2 MMA, 3 epilogue) if a wait ran out.
 // Needs K a multiple of 8 and 16-byte aligned operands.  scale_part (or null): the consuming end of a
 // carried norm, [M][scale_stride] with n_scale_part sums of squares a row over ``dim`` elements.
@@ -387,7 +388,7 @@ MV_API int mv_gemm_tc(const void* X, const void* W, const float* bias, void* out
                       int* err, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode == 3 && (N % 32 || ldo % 2)) return (int)cudaErrorInvalidValue;
+    if (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
     if (scale_part && (n_scale_part <= 0 || n_scale_part > scale_stride || dim <= 0)) return (int)cudaErrorInvalidValue;
     RowScale rs = {};
     if (scale_part) rs = RowScale{scale_part, n_scale_part, scale_stride, 1.0f / (float)dim, eps};
@@ -401,16 +402,17 @@ MV_API int mv_gemm_tc(const void* X, const void* W, const float* bias, void* out
 // The grouped product: the rows of X [M, K] are sorted by group and padded so that every tile of 128 rows belongs
 // to one group (tile_group [M / 128], negative for spare tiles); W [w_rows, w_cols] holds the groups' matrices one
 // below the other (b_row_step rows a group, b_k_step 0) or side by side along K (b_k_step columns a group, a
-// multiple of 8; b_row_step 0); N and K are ONE group's sizes.  Modes as mv_gemm_tc (no bias, no carried norm).
+// multiple of 8; b_row_step 0); N and K are ONE group's sizes.  Modes as mv_gemm_tc (no carried norm; bias, or mode 4's limits, are the
+// same for every group).
 // A tile's rows beyond its group's real rows hold whatever X holds there and give rows of ``out`` that nobody reads.
-MV_API int mv_gemm_tc_grouped(const void* X, const void* W, void* out, int mode, int M, int N, int K, int ldo,
+MV_API int mv_gemm_tc_grouped(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
                               int w_rows, int w_cols, const int* tile_group, int b_row_step, int b_k_step, int* err,
                               cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || M % BM || b_k_step % 8 || !tile_group || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
         return (int)cudaErrorInvalidValue;
-    if (mode == 3 && (N % 32 || ldo % 2)) return (int)cudaErrorInvalidValue;
+    if (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
     if (N <= 64)
-        return launch_grouped<64, 4>(X, W, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, b_k_step, err, stream);
-    return launch_grouped<128, 3>(X, W, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, b_k_step, err, stream);
+        return launch_grouped<64, 4>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, b_k_step, err, stream);
+    return launch_grouped<128, 3>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, b_k_step, err, stream);
 }

@@ -377,7 +377,7 @@ MV_API int mv_gemm_tc_pair(const void* X, const void* W, const float* bias, void
                            cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode == 3 && (N % 32 || ldo % 2)) return (int)cudaErrorInvalidValue;
+    if (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
     if (M <= BM || N < PAIR_BN / 2) return (int)cudaErrorInvalidValue;
     // an emitting product writes rows of 32 columns in 16-byte pieces: N in steps of 32, aligned buffers
     if (emit_x && (mode != 2 || ldo != N || N % 32 || !emit_g || !emit_part || emit_stride < (N + PAIR_BN - 1) / PAIR_BN ||

@@ -372,12 +372,12 @@ gemm_tc_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                     for (int e = 0; e < 4; ++e) v[e] *= sc;
                 }
-                if (bias) {
+                if (bias && mode != 4) {
 #pragma unroll
                     for (int e = 0; e < 4; ++e)
                         if (n + e < N) v[e] += bias[n + e];
                 }
-                if (mode == 3) {
+                if (mode >= 3) {
                     // rows in groups of 16 gate + 16 up: of every 8 lanes the first 4 hold gate rows,
                     // the next 4 the up rows of the same features
                     float up[4];
@@ -386,7 +386,9 @@ gemm_tc_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                     if ((lane & 4) == 0 && n + 16 < N) {
                         __nv_bfloat16* o = (__nv_bfloat16*)out + (size_t)m * ldo + (n >> 5) * 16 + (r & 15);
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) o[e] = __float2bfloat16_rn(v[e] / (1.0f + expf(-v[e])) * up[e]);
+                        for (int e = 0; e < 4; ++e)
+                            o[e] = __float2bfloat16_rn(mode == 4 ? mv_glu_clamped(v[e], up[e], bias[n], bias[N])
+                                                                 : mv_glu_silu(v[e], up[e]));
                     }
                 } else {
                     const size_t o = (size_t)m * ldo + n;
@@ -483,7 +485,7 @@ int launch(const void* X, const void* W, const float* bias, void* out, int mode,
 
 }  // namespace
 
-// Same contract as mv_gemm_small_m (modes 0-3, K a multiple of 8, 16-byte aligned operands;
+// Same contract as mv_gemm_small_m (modes 0-4, K a multiple of 8, 16-byte aligned operands;
 // scale_part / emit_x as there, with one sum per tile of 128 rows) for any M >= 1, plus the error
 // flag of the bounded waits.
 MV_API int mv_gemm_tc_swap(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N,
@@ -492,7 +494,7 @@ MV_API int mv_gemm_tc_swap(const void* X, const void* W, const float* bias, void
                            const void* next_w, long long next_bytes, int* err, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode == 3 && N % 32) return (int)cudaErrorInvalidValue;
+    if (mode >= 3 && (N % 32 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
     if (emit_x && (mode != 2 || ldo != N || !emit_g || !emit_part || emit_stride < (N + BM - 1) / BM))
         return (int)cudaErrorInvalidValue;
     if (scale_part && (n_scale_part <= 0 || n_scale_part > scale_stride || dim <= 0)) return (int)cudaErrorInvalidValue;

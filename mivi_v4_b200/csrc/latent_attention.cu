@@ -8,8 +8,10 @@
 //
 //   * latent_prepare: from a token's projections, the root-mean-square norm of c (with a weight), the rotation of
 //     r and of the queries' rotated parts (element i of the rotated part pairs with i + rot/2), the row into its page;
-//   * head_product: y[n, h, :] = W_h x[n, h, :] (or W_h^T), one small matrix per head: q -> qa and the output's way back
-//     (there with sigmoid(gate) on the result);
+//     where the queries come through a latent of their own, that latent's norm instead of their rotation;
+//   * head_product: y[n, h, :] = W_h x[n, h, :] (or W_h^T), one small matrix per head: q -> qa (there with the rotation
+//     of the queries' last elements, if latent_prepare has not done it) and the output's way back (there with
+//     sigmoid(gate) on the result, a gate an element or a head);
 //   * latent_attention: every query token on its own over its sequence's rows, causal, with a sliding window and a
 //     sink (a learned number per head whose exponential joins the softmax's denominator, with no value).
 // Scores, softmax, norms and angles are 32-bit; the cache is in the model's dtype.
@@ -22,14 +24,16 @@
 // ---------------------------------------------------------------------------------------------------- prepare
 // proj: 32-bit rows with stride ld; q at column q0: [head][dim unrotated | rot rotated]; the latent at column c0:
 // [rank | rot].  qa: 32-bit [N, nh, rank + rot]; its last rot columns are written here.  Of the rot elements the
-// first rot_dims turn (element i with i + rot_dims/2), the others pass unchanged.
+// first rot_dims turn (element i with i + rot_dims/2), the others pass unchanged.  cq (or null): the queries' own latent
+// at column cq0, over its root mean square and times wq, [N, q_rank] in the cache's dtype.
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(const float* __restrict__ proj, int ld, int q0, int c0, const float* __restrict__ wc, float eps,
                       const float* __restrict__ inv_freq, const int* __restrict__ positions,
                       const int* __restrict__ seq_of, const int* __restrict__ page_table, int table_stride,
                       int page_shift, T* __restrict__ pool, long long page_stride, float* __restrict__ qa, int nh, int dim,
-                      int rot, int rank, int rot_dims) {
+                      int rot, int rank, int rot_dims, int cq0, int q_rank, const float* __restrict__ wq,
+                      T* __restrict__ cq) {
     mv_pdl_begin();
     __shared__ float scratch[33];
     __shared__ float rot_sn[LA_MAX_ROT / 2], rot_cs[LA_MAX_ROT / 2];
@@ -61,6 +65,13 @@ latent_prepare_kernel(const float* __restrict__ proj, int ld, int q0, int c0, co
         }
         for (int i = rot_dims + threadIdx.x; i < rot; i += blockDim.x) dst[rank + i] = mv_from_f32<T>(r[i]);
     }
+    if (cq) {
+        const float* x = row + cq0;
+        float sq = 0.f;
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) sq = fmaf(x[i], x[i], sq);
+        const float qs = 1.0f / sqrtf(mv_block_sum(sq, scratch) / (float)q_rank + eps);
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) cq[(size_t)n * q_rank + i] = mv_from_f32<T>(x[i] * qs * wq[i]);
+    }
     if (!qa) return;                       // the queries are prepared elsewhere
     for (int e = threadIdx.x; e < nh * half; e += blockDim.x) {
         const int h = e / half, i = e - h * half;
@@ -81,18 +92,22 @@ MV_GUARD_SETTER(latent_attention)
 MV_API int mv_latent_prepare(const float* proj, int ld, int q0, int c0, const float* wc, float eps, const float* inv_freq,
                              const int* positions, const int* seq_of, const int* page_table, int table_stride,
                              int page_size, void* pool, long long page_stride, int dtype, float* qa, int N, int nh,
-                             int dim, int rot, int rank, int rot_dims, cudaStream_t stream) {
+                             int dim, int rot, int rank, int rot_dims, int cq0, int q_rank, const float* wq, void* cq,
+                             cudaStream_t stream) {
     if (N <= 0) return 0;
     if (rot < 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > rot || rot > LA_MAX_ROT || rank < 1 || page_size < 1 || (page_size & (page_size - 1)))
         return (int)cudaErrorInvalidValue;
+    if (cq && (q_rank < 1 || !wq)) return (int)cudaErrorInvalidValue;
     int shift = 0;
     while ((1 << shift) < page_size) ++shift;
     if (dtype == MV_DT_BF16)
         mv_launch(latent_prepare_kernel<__nv_bfloat16>, N, 256, 0, stream, proj, ld, q0, c0, wc, eps, inv_freq, positions,
-                  seq_of, page_table, table_stride, shift, (__nv_bfloat16*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims);
+                  seq_of, page_table, table_stride, shift, (__nv_bfloat16*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims, cq0,
+                  q_rank, wq, (__nv_bfloat16*)cq);
     else
         mv_launch(latent_prepare_kernel<float>, N, 256, 0, stream, proj, ld, q0, c0, wc, eps, inv_freq, positions, seq_of,
-                  page_table, table_stride, shift, (float*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims);
+                  page_table, table_stride, shift, (float*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims, cq0, q_rank, wq,
+                  (float*)cq);
     return mv_launch_status();
 }
 
@@ -100,21 +115,57 @@ MV_API int mv_latent_prepare(const float* proj, int ld, int q0, int c0, const fl
 // y[n, h, o] = sum_i W_h[o, i] x[n, h, i]  with W stored [nh * O, I] (head h owns rows h O .. (h + 1) O), or, with
 // `transposed`, W stored [nh * I, O] and y[n, h, o] = sum_i W_h[i, o] x[n, h, i].  x: 32-bit, element (n, h, i) at
 // x[n ldx + h hx + i]; y likewise with ldy, hy.  `gate` (or null): 32-bit logits, element (n, h, o) at
-// gate[n ldg + h O + o]; the result is multiplied by sigmoid of it.  Sums are 32-bit.
-// A block is 32 tokens x 64 outputs of one head; a thread has 2 tokens x 4 outputs.
+// gate[n ldg + h O + o], or with `gate_heads` (n, h) at gate[n ldg + h]; the result is multiplied by sigmoid of it.
+// Sums are 32-bit.  With tail.rot > 0 the rot elements after x's I are turned (see latent_prepare) and written after
+// y's O, by one more block along the grid's x.
+// A block is 32 tokens x 64 outputs of one head; a thread has 2 tokens x 4 outputs.  Steps of few tokens take the two
+// kernels after this one.
 #define HP_TN 32
 #define HP_TO 64
 #define HP_TK 32
 
+struct RotTail {
+    const float* inv_freq;
+    const int* positions;
+    int rot, rot_dims;
+};
+
+// the tail of tokens n0 .. n1 - 1 of head h: 32-bit in, 32-bit out (a tail is only asked for with 32-bit y)
+template <typename TY>
+__device__ __forceinline__ void rotate_tail(const RotTail& tail, const float* x, long long ldx, int hx, TY* y, long long ldy,
+                                            int hy, int h, int n0, int n1, int I, int O) {
+    const int half = tail.rot_dims >> 1;
+    for (int e = threadIdx.x; e < (n1 - n0) * tail.rot; e += blockDim.x) {
+        const int n = n0 + e / tail.rot, c = e % tail.rot;
+        const float* src = x + (size_t)n * ldx + (size_t)h * hx + I;
+        float v = src[c];
+        if (c < tail.rot_dims) {
+            float sn, cs;
+            sincosf((float)tail.positions[n] * tail.inv_freq[c < half ? c : c - half], &sn, &cs);
+            v = c < half ? v * cs - src[c + half] * sn : v * cs + src[c - half] * sn;
+        }
+        y[(size_t)n * ldy + (size_t)h * hy + O + c] = mv_from_f32<TY>(v);
+    }
+}
+
+__device__ __forceinline__ float head_gate(const float* gate, long long ldg, int gate_heads, int n, int h, int o, int O) {
+    if (!gate) return 1.f;
+    return 1.0f / (1.0f + expf(-gate[(size_t)n * ldg + (gate_heads ? (size_t)h : (size_t)h * O + o)]));
+}
+
 template <typename TW, typename TY>
 __global__ void __launch_bounds__(256)
 head_product_kernel(const float* __restrict__ x, long long ldx, int hx, const TW* __restrict__ w, int transposed,
-                    const float* __restrict__ gate, long long ldg, TY* __restrict__ y, long long ldy, int hy, int N, int I,
-                    int O) {
+                    const float* __restrict__ gate, long long ldg, int gate_heads, TY* __restrict__ y, long long ldy, int hy,
+                    int N, int I, int O, RotTail tail) {
     mv_pdl_begin();
     __shared__ float xs[HP_TN][HP_TK + 1];
     __shared__ float ws[HP_TK][HP_TO + 1];
     const int h = blockIdx.z, n0 = blockIdx.y * HP_TN, o0 = blockIdx.x * HP_TO;
+    if (o0 >= O) {
+        rotate_tail(tail, x, ldx, hx, y, ldy, hy, h, n0, min(N, n0 + HP_TN), I, O);
+        return;
+    }
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;       // outputs 4 tx .. 4 tx + 3, tokens 2 ty, 2 ty + 1
     float acc[2][4] = {};
     for (int k0 = 0; k0 < I; k0 += HP_TK) {
@@ -158,21 +209,168 @@ head_product_kernel(const float* __restrict__ x, long long ldx, int hx, const TW
             const int o = o0 + 4 * tx + j;
             if (o >= O) continue;
             float v = acc[t][j];
-            if (gate) v *= 1.0f / (1.0f + expf(-gate[(size_t)n * ldg + (size_t)h * O + o]));
+            if (gate) v *= head_gate(gate, ldg, gate_heads, n, h, o, O);
             y[(size_t)n * ldy + (size_t)h * hy + o] = mv_from_f32<TY>(v);
         }
     }
 }
 
+// Few tokens, the matrices transposed (W [nh * I, O]): a block is 8 tokens x 64 outputs of one head, a lane two
+// neighbouring outputs (consecutive lanes read consecutive elements of a row), the four warps a quarter of I each.
+#define HF_T 8
+#define HF_WARPS 4
+__device__ __forceinline__ void load2(const float* p, float& a, float& b) {
+    const float2 v = *reinterpret_cast<const float2*>(p);
+    a = v.x; b = v.y;
+}
+__device__ __forceinline__ void load2(const __nv_bfloat16* p, float& a, float& b) {
+    const unsigned v = *reinterpret_cast<const unsigned*>(p);
+    a = __uint_as_float(v << 16);
+    b = __uint_as_float(v & 0xffff0000u);
+}
+
+template <typename TW, typename TY>
+__global__ void __launch_bounds__(HF_WARPS * 32)
+head_product_few_t_kernel(const float* __restrict__ x, long long ldx, int hx, const TW* __restrict__ w,
+                          const float* __restrict__ gate, long long ldg, int gate_heads, TY* __restrict__ y, long long ldy,
+                          int hy, int N, int I, int O, RotTail tail) {
+    mv_pdl_begin();
+    extern __shared__ __align__(16) float hf_smem[];
+    float* xs = hf_smem;                                        // [I][HF_T]
+    __shared__ float sums[HF_WARPS][HF_T][64];
+    const int h = blockIdx.z, n0 = blockIdx.y * HF_T, o0 = blockIdx.x * 64;
+    const int nt = min(HF_T, N - n0);
+    if (o0 >= O) {
+        rotate_tail(tail, x, ldx, hx, y, ldy, hy, h, n0, n0 + nt, I, O);
+        return;
+    }
+    for (int e = threadIdx.x; e < I * HF_T; e += blockDim.x) {
+        const int t = e / I, i = e - t * I;
+        xs[i * HF_T + t] = t < nt ? x[(size_t)(n0 + t) * ldx + (size_t)h * hx + i] : 0.f;
+    }
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int per = (I + HF_WARPS - 1) / HF_WARPS, i0 = warp * per, i1 = min(I, i0 + per);
+    const int o = o0 + 2 * lane;
+    float a0[HF_T], a1[HF_T];
+#pragma unroll
+    for (int t = 0; t < HF_T; ++t) a0[t] = a1[t] = 0.f;
+    if (o < O) {
+        const TW* wp = w + (size_t)h * I * O + o;
+#pragma unroll 8
+        for (int i = i0; i < i1; ++i) {
+            float w0, w1;
+            load2(wp + (size_t)i * O, w0, w1);
+            const float4 xa = *reinterpret_cast<const float4*>(xs + i * HF_T), xb = *reinterpret_cast<const float4*>(xs + i * HF_T + 4);
+            const float xv[HF_T] = {xa.x, xa.y, xa.z, xa.w, xb.x, xb.y, xb.z, xb.w};
+#pragma unroll
+            for (int t = 0; t < HF_T; ++t) {
+                a0[t] = fmaf(w0, xv[t], a0[t]);
+                a1[t] = fmaf(w1, xv[t], a1[t]);
+            }
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < HF_T; ++t) {
+        sums[warp][t][2 * lane] = a0[t];
+        sums[warp][t][2 * lane + 1] = a1[t];
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < nt * 64; e += blockDim.x) {
+        const int t = e >> 6, c = e & 63;
+        if (o0 + c >= O) continue;
+        float v = 0.f;
+#pragma unroll
+        for (int k = 0; k < HF_WARPS; ++k) v += sums[k][t][c];
+        v *= head_gate(gate, ldg, gate_heads, n0 + t, h, o0 + c, O);
+        y[(size_t)(n0 + t) * ldy + (size_t)h * hy + o0 + c] = mv_from_f32<TY>(v);
+    }
+}
+
+// Few tokens, W [nh * O, I] (rows of whole 16-byte pieces): a block is 8 tokens x 16 outputs of one head, a warp four
+// outputs, a lane every 32nd piece of 8 elements of their rows; the 32 sums of a warp are folded while they are added,
+// so that lane l ends with the one of output l / 8 and token l % 8.
+template <typename TW, typename TY>
+__global__ void __launch_bounds__(HF_WARPS * 32)
+head_product_few_kernel(const float* __restrict__ x, long long ldx, int hx, const TW* __restrict__ w,
+                        const float* __restrict__ gate, long long ldg, int gate_heads, TY* __restrict__ y, long long ldy, int hy,
+                        int N, int I, int O) {
+    mv_pdl_begin();
+    extern __shared__ __align__(16) float hf_smem[];
+    float* xs = hf_smem;                                        // [HF_T][I]
+    const int h = blockIdx.z, n0 = blockIdx.y * HF_T;
+    const int nt = min(HF_T, N - n0);
+    for (int e = threadIdx.x; e < I * HF_T; e += blockDim.x) {
+        const int t = e / I, i = e - t * I;
+        xs[e] = t < nt ? x[(size_t)(n0 + t) * ldx + (size_t)h * hx + i] : 0.f;
+    }
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int o0 = blockIdx.x * 16 + warp * 4;
+    float acc[32];
+#pragma unroll
+    for (int k = 0; k < 32; ++k) acc[k] = 0.f;
+    for (int i = lane * 8; i < I; i += 256) {
+        float wv[4][8];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) mv_load8(w + ((size_t)h * O + min(o0 + k, O - 1)) * I + i, wv[k]);
+#pragma unroll
+        for (int t = 0; t < HF_T; ++t) {
+            float xv[8];
+            mv_load8(xs + t * I + i, xv);
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) acc[k * 8 + t] = fmaf(wv[k][e], xv[e], acc[k * 8 + t]);
+        }
+    }
+    // after the round with offset d a lane keeps the half of its sums whose index has bit d as its own lane number has
+#pragma unroll
+    for (int d = 16; d > 0; d >>= 1) {
+        const bool up = lane & d;
+#pragma unroll
+        for (int k = 0; k < d; ++k) {
+            const float give = up ? acc[k] : acc[k + d], keep = up ? acc[k + d] : acc[k];
+            acc[k] = keep + __shfl_xor_sync(0xffffffffu, give, d);
+        }
+    }
+    const int o = o0 + (lane >> 3), t = lane & 7;
+    if (o < O && t < nt)
+        y[(size_t)(n0 + t) * ldy + (size_t)h * hy + o] =
+            mv_from_f32<TY>(acc[0] * head_gate(gate, ldg, gate_heads, n0 + t, h, o, O));
+}
+
+#define HP_FEW_TOKENS 64
+#define HP_FEW_SMEM (40 * 1024)
+
+// gate: with gate_heads one logit a head.  rot > 0 (32-bit y, y's rows at least O + rot wide): the tail, see above.
 MV_API int mv_head_product(const float* x, long long ldx, int hx, const void* w, int w_dtype, int transposed,
-                           const float* gate, long long ldg, void* y, int y_dtype, long long ldy, int hy, int N, int nh,
-                           int I, int O, cudaStream_t stream) {
+                           const float* gate, long long ldg, int gate_heads, void* y, int y_dtype, long long ldy, int hy,
+                           int N, int nh, int I, int O, int rot, int rot_dims, const float* inv_freq, const int* positions,
+                           cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (nh < 1 || I < 1 || O < 1) return (int)cudaErrorInvalidValue;
-    const dim3 grid((O + HP_TO - 1) / HP_TO, (N + HP_TN - 1) / HP_TN, nh);
+    if (nh < 1 || I < 1 || O < 1 || rot < 0 || rot_dims < 0 || rot_dims > rot || rot_dims % 2 ||
+        (rot > 0 && (y_dtype != MV_DT_F32 || !positions || (rot_dims > 0 && !inv_freq))))
+        return (int)cudaErrorInvalidValue;
+    const RotTail tail = {inv_freq, positions, rot, rot_dims};
+    const int more = rot > 0 ? 1 : 0;
+    const size_t xs = sizeof(float) * (size_t)I * HF_T;
+    const size_t elt = w_dtype == MV_DT_BF16 ? 2 : 4;
+    const bool few = N <= HP_FEW_TOKENS && xs <= HP_FEW_SMEM && ((uintptr_t)w & 15) == 0;
+    const bool few_t = few && transposed && O % 2 == 0;
+    const bool few_n = few && !transposed && !more && (I * elt) % 16 == 0 && I % 8 == 0;
 #define HP_LAUNCH(TW, TY)                                                                                              \
-    mv_launch(head_product_kernel<TW, TY>, grid, 256, 0, stream, x, ldx, hx, (const TW*)w, transposed, gate, ldg, (TY*)y, \
-              ldy, hy, N, I, O)
+    do {                                                                                                               \
+        if (few_t)                                                                                                     \
+            mv_launch(head_product_few_t_kernel<TW, TY>, dim3((O + 63) / 64 + more, (N + HF_T - 1) / HF_T, nh),        \
+                      HF_WARPS * 32, xs, stream, x, ldx, hx, (const TW*)w, gate, ldg, gate_heads, (TY*)y, ldy, hy, N, I, O, tail); \
+        else if (few_n)                                                                                                \
+            mv_launch(head_product_few_kernel<TW, TY>, dim3((O + 15) / 16, (N + HF_T - 1) / HF_T, nh), HF_WARPS * 32,  \
+                      xs, stream, x, ldx, hx, (const TW*)w, gate, ldg, gate_heads, (TY*)y, ldy, hy, N, I, O);          \
+        else                                                                                                           \
+            mv_launch(head_product_kernel<TW, TY>, dim3((O + HP_TO - 1) / HP_TO + more, (N + HP_TN - 1) / HP_TN, nh), 256, 0, \
+                      stream, x, ldx, hx, (const TW*)w, transposed, gate, ldg, gate_heads, (TY*)y, ldy, hy, N, I, O, tail); \
+    } while (0)
     if (w_dtype == MV_DT_BF16) {
         if (y_dtype == MV_DT_BF16) HP_LAUNCH(__nv_bfloat16, __nv_bfloat16); else HP_LAUNCH(__nv_bfloat16, float);
     } else {

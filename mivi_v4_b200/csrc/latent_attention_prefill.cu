@@ -51,6 +51,7 @@ __device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const void* 
 __device__ __forceinline__ int first_seen(int start, int window) { return window > 0 ? max(0, start - window + 1) : 0; }
 
 // ------------------------------------------------------------------------------------------------------ queries
+#define LQ_MAX_ROT 512
 __global__ void __launch_bounds__(256)
 latent_query_kernel(const float* __restrict__ proj, int ld, int q0, const float* __restrict__ inv_freq,
                     const int* __restrict__ positions, __nv_bfloat16* __restrict__ q, int nh, int dim, int rot,
@@ -59,7 +60,9 @@ latent_query_kernel(const float* __restrict__ proj, int ld, int q0, const float*
     const int n = blockIdx.x;
     const int dk = dim + rot, half = rot_dims >> 1;
     const float* row = proj + (size_t)n * ld + q0;
-    const float pos = (float)positions[n];
+    __shared__ float sn_s[LQ_MAX_ROT / 2], cs_s[LQ_MAX_ROT / 2];          // a token's angles, once for all heads
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)positions[n] * inv_freq[i], &sn_s[i], &cs_s[i]);
+    __syncthreads();
     __nv_bfloat16* dst = q + (size_t)n * nh * dk;
     for (int e = threadIdx.x; e < nh * dk; e += blockDim.x) {
         const int c = e % dk;
@@ -67,9 +70,7 @@ latent_query_kernel(const float* __restrict__ proj, int ld, int q0, const float*
         float x = row[e];
         if (i >= 0 && i < rot_dims) {
             const int f = i < half ? i : i - half;
-            float sn, cs;
-            sincosf(pos * inv_freq[f], &sn, &cs);
-            x = i < half ? x * cs - row[e + half] * sn : x * cs + row[e - half] * sn;
+            x = i < half ? x * cs_s[f] - row[e + half] * sn_s[f] : x * cs_s[f] + row[e - half] * sn_s[f];
         }
         dst[e] = __float2bfloat16(x);
     }
@@ -104,7 +105,7 @@ latent_gather_kernel(const __nv_bfloat16* __restrict__ pool, long long page_stri
 
 // ---------------------------------------------------------------------------------------------------- attention
 // q [N, nh, dim + rot]; kx [rows, ld_kx]: head h's unrotated keys at column h dim, its values at v0 + h dv; r [rows, rot];
-// gate: 32-bit logits [N, >= nh dv] with row stride ld_gate, or null; o [N, nh dv].  The softmax weights enter the
+// gate: 32-bit logits [N, >= nh dv] with row stride ld_gate (with gate_heads [N, >= nh], one a head), or null; o [N, nh dv].  The softmax weights enter the
 // second product as two bfloat16 numbers each (the rounded weight and what the rounding left), so the sum over the
 // values carries the weights to 16 bits of mantissa although the tensor cores read bfloat16.
 template <int DKM, int DVM>
@@ -112,7 +113,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
 latent_attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kx, int ld_kx,
                                 int v0, const __nv_bfloat16* __restrict__ rk, const int* __restrict__ cu,
                                 const int* __restrict__ starts, const float* __restrict__ sinks,
-                                const float* __restrict__ gate, int ld_gate, __nv_bfloat16* __restrict__ o, int B, int nh,
+                                const float* __restrict__ gate, int ld_gate, int gate_heads, __nv_bfloat16* __restrict__ o, int B, int nh,
                                 int dim, int rot, int dv, float scale, int window) {
     mv_pdl_begin();
     const int dk = dim + rot;
@@ -293,12 +294,13 @@ latent_attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_
     for (int half = 0; half < 2; ++half) {
         if (qi[half] >= nq) continue;
         const size_t n = (size_t)(row0 + qi[half]);
-        const float* g = gate ? gate + n * ld_gate + (size_t)h * dv + 2 * t4 : nullptr;
+        const float* g = gate && !gate_heads ? gate + n * ld_gate + (size_t)h * dv + 2 * t4 : nullptr;
+        const float gh = (gate && gate_heads ? 1.0f / (1.0f + expf(-gate[n * ld_gate + h])) : 1.f) * inv[half];
         __nv_bfloat16* dst = o + (n * nh + h) * dv + 2 * t4;
 #pragma unroll
         for (int j = 0; j < DVM / 8; ++j) {
             if (j * 8 < dv) {
-                float x = oacc[j][2 * half] * inv[half], y = oacc[j][2 * half + 1] * inv[half];
+                float x = oacc[j][2 * half] * gh, y = oacc[j][2 * half + 1] * gh;
                 if (g) {
                     x *= 1.0f / (1.0f + expf(-g[j * 8]));
                     y *= 1.0f / (1.0f + expf(-g[j * 8 + 1]));
@@ -311,7 +313,7 @@ latent_attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_
 
 template <int DKM, int DVM>
 int launch(const void* q, const void* kx, int ld_kx, int v0, const void* rk, const int* cu, const int* starts,
-           const float* sinks, const float* gate, int ld_gate, void* o, int N, int B, int nh, int dim, int rot, int dv,
+           const float* sinks, const float* gate, int ld_gate, int gate_heads, void* o, int N, int B, int nh, int dim, int rot, int dv,
            float scale, int window, cudaStream_t stream) {
     const size_t smem = (size_t)2 * KB * (dim + rot + 8 + dv + 8) * sizeof(__nv_bfloat16);
     static bool attr_set = false;
@@ -323,7 +325,7 @@ int launch(const void* q, const void* kx, int ld_kx, int v0, const void* rk, con
     const dim3 grid((N + QT - 1) / QT + B, nh);       // an upper bound of the tiles; spare blocks return at once
     mv_launch(latent_attention_prefill_kernel<DKM, DVM>, grid, NWARPS * 32, smem, stream, (const __nv_bfloat16*)q,
               (const __nv_bfloat16*)kx, ld_kx, v0, (const __nv_bfloat16*)rk, cu, starts, sinks, gate, ld_gate,
-              (__nv_bfloat16*)o, B, nh, dim, rot, dv, scale, window);
+              gate_heads, (__nv_bfloat16*)o, B, nh, dim, rot, dv, scale, window);
     return mv_launch_status();
 }
 
@@ -336,7 +338,7 @@ MV_GUARD_SETTER(latent_attention_prefill)
 MV_API int mv_latent_query(const float* proj, int ld, int q0, const float* inv_freq, const int* positions, void* q, int N,
                            int nh, int dim, int rot, int rot_dims, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (rot_dims < 0 || rot_dims > rot || (rot_dims & 1) || (rot_dims && !inv_freq)) return (int)cudaErrorInvalidValue;
+    if (rot_dims < 0 || rot_dims > rot || rot_dims > LQ_MAX_ROT || (rot_dims & 1) || (rot_dims && !inv_freq)) return (int)cudaErrorInvalidValue;
     mv_launch(latent_query_kernel, N, 256, 0, stream, proj, ld, q0, inv_freq, positions, (__nv_bfloat16*)q, nh, dim, rot,
               rot_dims);
     return mv_launch_status();
@@ -358,7 +360,8 @@ MV_API int mv_latent_gather(const void* pool, long long page_stride, const int* 
 
 // bfloat16; dim and rot multiples of 8 whose sum is a multiple of 16 up to 192; dv a multiple of 16 up to 128.
 MV_API int mv_latent_attention_prefill(const void* q, const void* kx, int ld_kx, int v0, const void* r, const int* cu,
-                                       const int* starts, const float* sinks, const float* gate, int ld_gate, void* o,
+                                       const int* starts, const float* sinks, const float* gate, int ld_gate,
+                                       int gate_heads, void* o,
                                        int N, int B, int nh, int dim, int rot, int dv, float scale, int window,
                                        cudaStream_t stream) {
     if (N <= 0) return 0;
@@ -367,7 +370,7 @@ MV_API int mv_latent_attention_prefill(const void* q, const void* kx, int ld_kx,
         window < 0)
         return (int)cudaErrorInvalidValue;
 #define LP_GO(A, C)                                                                                                        \
-    return launch<A, C>(q, kx, ld_kx, v0, r, cu, starts, sinks, gate, ld_gate, o, N, B, nh, dim, rot, dv, scale, window, \
+    return launch<A, C>(q, kx, ld_kx, v0, r, cu, starts, sinks, gate, ld_gate, gate_heads, o, N, B, nh, dim, rot, dv, scale, window, \
                         stream)
     if (dk <= 128 && dv <= 64) LP_GO(128, 64);
     if (dk <= 128) LP_GO(128, 128);

@@ -1,11 +1,12 @@
 // Routing of a mixture of experts, and the gated activation of the chosen experts.
 //
-// Router: s_e = sigmoid(z_e) from 32-bit logits, or softmax over all of them; a correction per expert may be added
+// Router: s_e = sigmoid(z_e) from 32-bit logits (a bias may be added to them first), or softmax over all of them, or
+// the logits themselves with weights softmax(the chosen logits); a correction per expert may be added
 // for the choice alone; some of the routed entries may be identity experts (no matrices: their output is their input).  The experts form `n_groups` equal groups of neighbours; a
 // group's score is the sum of its two largest s (of its only one, in groups of one); only experts of the
 // `keep` best groups can be chosen; the `top` largest s among those are chosen; their weights are s divided
 // by the sum of the chosen s (+ 1e-20).  Ties go to the lower index.  A shared expert's gate, sigmoid of one
-// more logit, is written as one more column.  All of it is 32-bit.
+// more logit, is written as one more column (a shared expert without a gate has none).  All of it is 32-bit.
 //
 // Output: a dense row of weights per token, [experts (+ 1)], zero for the experts that were not chosen, and
 // the chosen experts with their weights as lists [top].
@@ -22,14 +23,15 @@ __device__ __forceinline__ void re_argmax(float& v, int& i) {
     }
 }
 
-// one warp a token.  mode 0: scores sigmoid(z); mode 1: scores softmax(z) over all E routed entries.  `correction`
+// one warp a token.  z <- z + bias (or null).  mode 0: scores sigmoid(z); mode 1: scores softmax(z) over all E routed
+// entries; mode 2: scores z, the weights are softmax over the chosen z alone, times out_scale.  `correction`
 // (or null) is added to the scores for the CHOICE only; the weights are the chosen entries' own scores over their sum
 // (+ 1e-20), times out_scale.  The last n_identity of the E entries are identity experts: the dense row is laid out
 // [E - n_identity experts | the shared gate, if any | n_identity identity weights].
 __global__ void __launch_bounds__(128)
 route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int* __restrict__ pick,
              float* __restrict__ pick_w, int N, int E, int n_groups, int keep, int top, int shared_gate, int mode,
-             const float* __restrict__ correction, float out_scale, int n_identity) {
+             const float* __restrict__ correction, float out_scale, int n_identity, const float* __restrict__ bias) {
     mv_pdl_begin();
     extern __shared__ float re_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -43,21 +45,22 @@ route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int
     const int n_real = E - n_identity, sg = shared_gate ? 1 : 0;
     const int cols = E + sg;
     float* dr = dense + (size_t)n * cols;
+    for (int e = lane; e < E; e += 32) s[e] = zr[e] + (bias ? bias[e] : 0.f);       // a lane's own entries
     if (mode == 1) {
         float mx = NEG;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zr[e]);
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, s[e]);
         mx = mv_warp_max(mx);
         float sum = 0.f;
         for (int e = lane; e < E; e += 32) {
-            const float v = expf(zr[e] - mx);
+            const float v = expf(s[e] - mx);
             s[e] = v;
             sum += v;
         }
         sum = mv_warp_sum(sum);
         const float inv = 1.0f / sum;
         for (int e = lane; e < E; e += 32) s[e] *= inv;
-    } else {
-        for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-zr[e]));
+    } else if (mode == 0) {
+        for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
     }
     for (int e = lane; e < E; e += 32) ch[e] = s[e] + (correction ? correction[e] : 0.f);
     for (int c = lane; c < cols; c += 32) dr[c] = 0.f;
@@ -87,7 +90,7 @@ route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int
             if (gs[e / per] != 2.f * NEG) ch[e] = NEG;
         __syncwarp();
     }
-    float sum = 0.f;
+    float sum = 0.f, best = NEG;
     for (int r = 0; r < top; ++r) {
         float v = NEG; int i = 0x7fffffff;
         for (int e = lane; e < E; e += 32)
@@ -95,6 +98,7 @@ route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int
         re_argmax(v, i);
         const float sc = s[i];
         sum += sc;
+        best = fmaxf(best, sc);
         if (lane == 0) {
             pick[(size_t)n * top + r] = i;
             pick_w[(size_t)n * top + r] = sc;
@@ -102,28 +106,32 @@ route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int
         }
         __syncwarp();
     }
-    const float inv = out_scale / (sum + 1e-20f);
+    // (top <= 32 is checked by the host)
+    float w = lane < top ? pick_w[(size_t)n * top + lane] : 0.f;
+    if (mode == 2) {
+        w = lane < top ? expf(w - best) : 0.f;
+        sum = mv_warp_sum(w);
+    }
+    w *= out_scale / (mode == 2 ? sum : sum + 1e-20f);
     if (lane < top) {
-        // (top <= 32 is checked by the host)
-        const float w = pick_w[(size_t)n * top + lane] * inv;
         pick_w[(size_t)n * top + lane] = w;
         const int i = pick[(size_t)n * top + lane];
         dr[i < n_real ? i : i + sg] = w;
     }
 }
 
-// z [N, >= E (+ 1)] with row stride ld; dense [N, E (+ 1)]; pick, pick_w [N, top]; correction [E] or null.
+// z [N, >= E (+ 1)] with row stride ld; dense [N, E (+ 1)]; pick, pick_w [N, top]; correction, bias [E] or null.
 MV_API int mv_route(const float* z, int ld, float* dense, int* pick, float* pick_w, int N, int E, int n_groups,
                     int keep, int top, int shared_gate, int mode, const float* correction, float out_scale,
-                    int n_identity, cudaStream_t stream) {
+                    int n_identity, const float* bias, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (E < 1 || E > RE_MAX_EXPERTS || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups || top < 1 ||
-        top > 32 || top > keep * (E / n_groups) || n_identity < 0 || n_identity > E || mode < 0 || mode > 1)
+        top > 32 || top > keep * (E / n_groups) || n_identity < 0 || n_identity > E || mode < 0 || mode > 2)
         return (int)cudaErrorInvalidValue;
     const int warps = 4;
     const size_t smem = sizeof(float) * warps * (size_t)(2 * E + n_groups);
     mv_launch(route_kernel, (N + warps - 1) / warps, warps * 32, smem, stream, z, ld, dense, pick, pick_w, N, E,
-              n_groups, keep, top, shared_gate, mode, correction, out_scale, n_identity);
+              n_groups, keep, top, shared_gate, mode, correction, out_scale, n_identity, bias);
     return mv_launch_status();
 }
 
@@ -157,47 +165,50 @@ MV_API int mv_identity_experts(const void* h, int dtype, const float* dense, int
 }
 
 // ------------------------------------------------------------------------------------------------
-// hid[n, c] = w[n, expert(c)] * silu(gate[n, c]) * up[n, c] over the columns of all experts laid end to end
+// hid[n, c] = w[n, expert(c)] * act(gate[n, c], up[n, c]) (silu(gate) * up, or with `limit` > 0 the clamped gated
+// activation with that limit, `shared_limit` for the shared expert, and `alpha`) over the columns of all experts laid end to end
 // (expert e owns [e * ff, (e + 1) * ff), a shared expert the `shared_ff` columns after them, with the weight of
-// column E).  gu [N, 2 * F] holds an expert's gates and ups together, [e * 2 ff, (e + 1) * 2 ff): alternating in
+// column E, or 1 where it has no gate).  gu [N, 2 * F] holds an expert's gates and ups together, [e * 2 ff, (e + 1) * 2 ff): alternating in
 // groups of 16 columns (16 gates, their 16 ups, ...) where `group` says so, else the gates, then the ups; the
 // shared expert's block follows with `shared_group`.  Where the weight is zero nothing is computed.
 template <typename TO>
 __global__ void __launch_bounds__(256)
 routed_glu_kernel(const float* __restrict__ gu, const float* __restrict__ dense, TO* __restrict__ hid, long long total,
-                  int F, int E, int ff, int shared_ff, int cols, int group, int shared_group) {
+                  int F, int E, int ff, int shared_ff, int cols, int group, int shared_group, int shared_gate, float limit,
+                  float shared_limit, float alpha) {
     mv_pdl_begin();
     const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
     const long long n = idx / F;
     const int c = (int)(idx - n * F);
     const int e = c < E * ff ? c / ff : E;
-    const float w = dense[n * cols + e];
+    const float w = e < E || shared_gate ? dense[n * cols + e] : 1.f;
     float out = 0.f;
     if (w != 0.f) {
         const int cc = c - e * ff, width = e < E ? ff : shared_ff, grp = e < E ? group : shared_group;
         const float* blk = gu + n * 2 * F + (size_t)e * 2 * ff;
         const int gi = grp ? (cc / grp) * 2 * grp + cc % grp : cc;
         const float g = blk[gi], u = blk[gi + (grp ? grp : width)];
-        out = w * (g / (1.0f + expf(-g))) * u;
+        out = w * (limit > 0.f ? mv_glu_clamped(g, u, e < E ? limit : shared_limit, alpha) : mv_glu_silu(g, u));
     }
     hid[idx] = mv_from_f32<TO>(out);
 }
 
 // extra_cols: columns of a dense row after the experts' (and the shared gate's) that belong to others
 MV_API int mv_routed_glu(const float* gu, const float* dense, void* hid, int hid_dtype, int N, int E, int ff,
-                         int shared_ff, int group, int shared_group, int extra_cols, cudaStream_t stream) {
+                         int shared_ff, int group, int shared_group, int extra_cols, int shared_gate, float limit,
+                         float shared_limit, float alpha, cudaStream_t stream) {
     if (N <= 0) return 0;
-    const int F = E * ff + shared_ff, cols = E + (shared_ff ? 1 : 0) + extra_cols;
+    const int F = E * ff + shared_ff, cols = E + (shared_ff && shared_gate ? 1 : 0) + extra_cols;
     if ((group && ff % group) || (shared_group && shared_ff % shared_group)) return (int)cudaErrorInvalidValue;
     const long long total = (long long)N * F;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (hid_dtype == MV_DT_BF16)
         mv_launch(routed_glu_kernel<__nv_bfloat16>, blocks, 256, 0, stream, gu, dense, (__nv_bfloat16*)hid, total, F, E,
-                  ff, shared_ff, cols, group, shared_group);
+                  ff, shared_ff, cols, group, shared_group, shared_gate, limit, shared_limit, alpha);
     else
         mv_launch(routed_glu_kernel<float>, blocks, 256, 0, stream, gu, dense, (float*)hid, total, F, E, ff, shared_ff, cols,
-                  group, shared_group);
+                  group, shared_group, shared_gate, limit, shared_limit, alpha);
     return mv_launch_status();
 }
 
@@ -346,12 +357,13 @@ MV_API int mv_expert_combine(const float* ys, const int* place, const float* pic
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
 scale_expert_columns_kernel(T* __restrict__ h, const float* __restrict__ dense, long long total, int F, int E, int ff,
-                            int cols) {
+                            int cols, int shared_gate) {
     mv_pdl_begin();
     const long long idx = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (idx >= total) return;
     const long long n = idx / F;
     const int c = (int)(idx - n * F);
+    if (c >= E * ff && !shared_gate) return;                   // a shared expert without a gate: as it is
     const float w = dense[n * cols + (c < E * ff ? c / ff : E)];
     if (V == 8) {
         float x[8];
@@ -364,13 +376,13 @@ scale_expert_columns_kernel(T* __restrict__ h, const float* __restrict__ dense, 
 }
 
 MV_API int mv_scale_expert_columns(void* h, int dtype, const float* dense, int N, int E, int ff, int shared_ff,
-                                   int extra_cols, cudaStream_t stream) {
+                                   int extra_cols, int shared_gate, cudaStream_t stream) {
     if (N <= 0) return 0;
-    const int F = E * ff + shared_ff, cols = E + (shared_ff ? 1 : 0) + extra_cols;
+    const int F = E * ff + shared_ff, cols = E + (shared_ff && shared_gate ? 1 : 0) + extra_cols;
     const long long total = (long long)N * F;
     const bool wide = ff % 8 == 0 && shared_ff % 8 == 0 && ((uintptr_t)h % 16) == 0;
     const unsigned blocks = (unsigned)((total / (wide ? 8 : 1) + 255) / 256);
-#define SE_LAUNCH(T, V) mv_launch(scale_expert_columns_kernel<T, V>, blocks, 256, 0, stream, (T*)h, dense, total, F, E, ff, cols)
+#define SE_LAUNCH(T, V) mv_launch(scale_expert_columns_kernel<T, V>, blocks, 256, 0, stream, (T*)h, dense, total, F, E, ff, cols, shared_gate)
     if (dtype == MV_DT_BF16) { if (wide) SE_LAUNCH(__nv_bfloat16, 8); else SE_LAUNCH(__nv_bfloat16, 1); }
     else { if (wide) SE_LAUNCH(float, 8); else SE_LAUNCH(float, 1); }
 #undef SE_LAUNCH

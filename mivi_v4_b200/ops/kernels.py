@@ -49,7 +49,8 @@ _SIGNATURES = {
         "mv_gated_rmsnorm": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _F, _I, _P],
         "mv_rmsnorm_add": [_P, _P, _P, _I, _I, _F, _P],
         "mv_rmsnorm_add_layernorm": [_P, _P, _F, _P, _P, _F, _P, _I, _I, _I, _P],
-        "mv_glu_clamped": [_P, _P, _I, _I, _I, _F, _F, _P],
+        "mv_glu_clamped": [_P, _P, _I, _I, _I, _I, _F, _F, _P],
+        "mv_sum_norm": [_P, _F, _P, _F, _P, _Q, _P, _P, _F, _P, _F, _P, _I, _I, _I, _P],
         "mv_table_gate": [_P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _P],
         "mv_table_gate_proj": [_P, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _P],
         "mv_round_rows": [_P, _P, _I, _Q, _P],
@@ -77,14 +78,15 @@ _SIGNATURES = {
         "mv_causal_conv": [_P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
         "mv_ssm_decode_prepare": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
         "mv_step_size": [_P, _I, _P, _P, _P, _P, _I, _I, _P],
-        "mv_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _P],
-        "mv_routed_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
-        "mv_scale_expert_columns": [_P, _I, _P, _I, _I, _I, _I, _I, _P],
+        "mv_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _P, _P],
+        "mv_routed_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
+        "mv_scale_expert_columns": [_P, _I, _P, _I, _I, _I, _I, _I, _I, _P],
         "mv_identity_experts": [_P, _I, _P, _I, _I, _I, _P, _I, _I, _I, _P],
-        "mv_embed_bigram": [_P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _Q, _Q, _P],
+        "mv_embed_bigram": [_P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _Q, _Q, _P],
         "mv_add_rows_vector": [_P, _P, _P, _I, _I, _P],
-        "mv_latent_prepare": [_P, _I, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _P, _Q, _I, _P, _I, _I, _I, _I, _I, _I, _P],
-        "mv_head_product": [_P, _Q, _I, _P, _I, _I, _P, _Q, _P, _I, _Q, _I, _I, _I, _I, _I, _P],
+        "mv_latent_prepare": [_P, _I, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _P, _Q, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I,
+                              _P, _P, _P],
+        "mv_head_product": [_P, _Q, _I, _P, _I, _I, _P, _Q, _I, _P, _I, _Q, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P],
         "mv_latent_attention": [_P, _P, _Q, _I, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P],
         "mv_delta_scan_long": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _F, _F, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
         "mv_delta_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _F, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
@@ -101,7 +103,7 @@ _SIGNATURES = {
         "mv_gemm_small_m_heads": [_P, _P, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _Q, _P, _I, _I, _I, _I,
                                   _P, _I, _I, _I, _F, _P, _Q, _P],
         "mv_gemm_tc": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P],
-        "mv_gemm_tc_grouped": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P],
+        "mv_gemm_tc_grouped": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P],
         "mv_gemm_tc_pair": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P, _P, _I, _P, _P],
         "mv_gemm_tc_swap": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P, _P, _I, _P, _Q, _P, _P],
         "mv_gemm_tc_swap_shortconv": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _Q,
@@ -115,7 +117,7 @@ _SIGNATURES = {
         "mv_attention_prefill_tc": [_P, _P, _Q, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
         "mv_latent_query": [_P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "mv_latent_gather": [_P, _Q, _P, _I, _I, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P],
-        "mv_latent_attention_prefill": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P],
+        "mv_latent_attention_prefill": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P],
     },
 }
 _fns = {}
@@ -447,13 +449,15 @@ def rmsnorm_add_layernorm(y: torch.Tensor, w: torch.Tensor, eps: float, resid: t
     return out
 
 
-def glu_clamped(gu: torch.Tensor, out: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+def glu_clamped(gu: torch.Tensor, out: torch.Tensor, limit: float, alpha: float, group: int = 0) -> torch.Tensor:
     """out = g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); gate and
-    up are the two halves of a row of ``gu`` (float32)."""
+    up are the two halves of a row of ``gu`` (float32), or alternate in groups of ``group`` columns."""
     N, F2 = gu.shape
     F = F2 // 2
+    if group and F % group:
+        raise KernelError(f"glu_clamped: width {F} is not a multiple of the group size {group}")
     _check(_fn("core", "mv_glu_clamped")(
-        _need(gu, "glu in", torch.float32, (N, 2 * F)), _need(out, "glu out", None, (N, F)), _dt(out), N, F,
+        _need(gu, "glu in", torch.float32, (N, 2 * F)), _need(out, "glu out", None, (N, F)), _dt(out), N, F, int(group),
         float(limit), float(alpha), _stream()), "mv_glu_clamped")
     account(_nbytes(gu, out))
     return out
@@ -546,6 +550,25 @@ def rmsnorm_add_sum(y1: torch.Tensor, w: torch.Tensor, eps: float, resid: torch.
         _need(resid, "residual stream", torch.float32, (N, H)), _need(rounded, "rounded rows", None, (N, H), True),
         _dt(rounded) if rounded is not None else F32, N, H, float(eps), _stream()), "mv_rmsnorm_add_sum")
     account(N * H * (12 + (4 if y2 is not None else 0) + (rounded.element_size() if rounded is not None else 0)))
+    return resid
+
+
+def sum_norm(y1: torch.Tensor, resid: torch.Tensor, alpha: float, w: torch.Tensor, eps: float, *, s1: float = 1.0,
+             y2: Optional[torch.Tensor] = None, s2: float = 1.0, gate: Optional[torch.Tensor] = None,
+             gate_bias: Optional[torch.Tensor] = None, rounded: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The norm after the residual sum: x = alpha * resid + sigmoid(gate + gate_bias) * (s1 y1 + s2 y2) (``gate`` None:
+    no factor; ``y2`` None: s1 y1), then resid = x / sqrt(mean(x^2) + eps) * w, all float32; ``rounded`` also gets the
+    completed rows in its own dtype.  ``gate`` [N, H] may be a column slice of a wider matrix."""
+    N, H = resid.shape
+    gp, ldg = _cols(gate, "sum_norm gate", N, H) if gate is not None else (None, 0)
+    _check(_fn("core", "mv_sum_norm")(
+        _need(y1, "sum_norm y1", torch.float32, (N, H)), float(s1), _need(y2, "sum_norm y2", torch.float32, (N, H), True),
+        float(s2), gp, ldg, _need(gate_bias, "gate bias", torch.float32, (H,), True), _need(resid, "residual stream", torch.float32),
+        float(alpha), _need(w, "norm weight", torch.float32, (H,)), float(eps),
+        _need(rounded, "rounded rows", None, (N, H), True), _dt(rounded) if rounded is not None else F32, N, H, _stream()),
+        "mv_sum_norm")
+    account(N * H * (12 + (4 if y2 is not None else 0) + (4 if gate is not None else 0)
+                     + (rounded.element_size() if rounded is not None else 0)))
     return resid
 
 
@@ -751,14 +774,17 @@ def ssm_decode_prepare(u: torch.Tensor, taps: torch.Tensor, bias: Optional[torch
 MAX_EXPERTS = 1024
 
 
-ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
+ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_CHOSEN_SOFTMAX = 0, 1, 2
 
 
 def route(z: torch.Tensor, dense: torch.Tensor, pick: torch.Tensor, pick_w: torch.Tensor, n_experts: int,
           n_groups: int, keep: int, top: int, shared_gate: bool, *, mode: int = ROUTE_SIGMOID,
-          correction: Optional[torch.Tensor] = None, out_scale: float = 1.0, n_identity: int = 0) -> None:
-    """Router of a mixture of experts from float32 logits ``z`` [N, routed (+ 1)]: scores sigmoid(z), or with
-    ``ROUTE_SOFTMAX`` softmax(z) over all routed entries; the entries
+          correction: Optional[torch.Tensor] = None, out_scale: float = 1.0, n_identity: int = 0,
+          bias: Optional[torch.Tensor] = None) -> None:
+    """Router of a mixture of experts from float32 logits ``z`` [N, routed (+ 1)] (``bias`` [routed] is added to them
+    first): scores sigmoid(z), or with ``ROUTE_SOFTMAX`` softmax(z) over all routed entries, or with
+    ``ROUTE_CHOSEN_SOFTMAX`` the logits themselves, the weights then being softmax over the chosen logits alone, times
+    ``out_scale``; the entries
     form ``n_groups`` equal groups of neighbours whose score is the sum of their two largest scores; among the
     entries of the ``keep`` best groups the ``top`` largest are chosen, with weights score / (sum of the chosen
     scores + 1e-20) * ``out_scale``.  ``correction`` [routed] is added to the scores for the choice only.
@@ -777,7 +803,7 @@ def route(z: torch.Tensor, dense: torch.Tensor, pick: torch.Tensor, pick_w: torc
         zp, ldz, _need(dense, "route weights", torch.float32, (N, cols)), _need(pick, "route picks", torch.int32, (N, top)),
         _need(pick_w, "route pick weights", torch.float32, (N, top)), N, E, int(n_groups), int(keep), int(top),
         int(bool(shared_gate)), int(mode), _need(correction, "route correction", torch.float32, (E,), True),
-        float(out_scale), int(n_identity), _stream()), "mv_route")
+        float(out_scale), int(n_identity), _need(bias, "router bias", torch.float32, (E,), True), _stream()), "mv_route")
     account(N * cols * 8)
 
 
@@ -797,12 +823,15 @@ def identity_experts(h: torch.Tensor, dense: torch.Tensor, col0: int, n_cols: in
 
 
 def routed_glu(gu: torch.Tensor, dense: torch.Tensor, hid: torch.Tensor, n_experts: int, ff: int, shared_ff: int,
-               group: int = 0, shared_group: int = 0, extra_cols: int = 0) -> torch.Tensor:
+               group: int = 0, shared_group: int = 0, extra_cols: int = 0, shared_gate: bool = True, limit: float = 0.0,
+               shared_limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """hid[n, c] = weight(n, expert of column c) * silu(gate[n, c]) * up[n, c] over the columns of all experts end to
     end (then a shared expert's), from ``gu`` [N, 2 * F] float32 and the router's dense weights; nothing is computed
     where the weight is zero.  ``gu`` holds each expert's gates and ups together, [e * 2 ff, (e + 1) * 2 ff): the gates,
     then the ups, or with ``group`` 16 alternating in groups of 16 columns; the shared expert's block likewise with
-    ``shared_group``."""
+    ``shared_group``.  Without ``shared_gate`` the dense weights have no column for the shared expert and its weight
+    is 1.  ``limit`` > 0: the clamped gated activation of :func:`glu_clamped` instead of silu(gate) * up, with
+    ``shared_limit`` for the shared expert."""
     N, F = hid.shape
     if F != n_experts * ff + shared_ff:
         raise KernelError(f"routed_glu: {F} columns for {n_experts} experts of {ff} and a shared one of {shared_ff}")
@@ -810,24 +839,25 @@ def routed_glu(gu: torch.Tensor, dense: torch.Tensor, hid: torch.Tensor, n_exper
         raise KernelError(f"routed_glu: widths {ff} and {shared_ff} against groups of {group} and {shared_group}")
     _check(_fn("core", "mv_routed_glu")(
         _need(gu, "routed_glu input", torch.float32, (N, 2 * F)),
-        _need(dense, "route weights", torch.float32, (N, n_experts + (1 if shared_ff else 0) + extra_cols)),
+        _need(dense, "route weights", torch.float32, (N, n_experts + (1 if shared_ff and shared_gate else 0) + extra_cols)),
         _need(hid, "routed_glu out"), _dt(hid), N, int(n_experts), int(ff), int(shared_ff), int(group), int(shared_group),
-        int(extra_cols), _stream()), "mv_routed_glu")
+        int(extra_cols), int(bool(shared_gate)), float(limit), float(shared_limit), float(alpha), _stream()), "mv_routed_glu")
     account(N * F * (8 + hid.element_size()))
     return hid
 
 
 def scale_expert_columns(h: torch.Tensor, dense: torch.Tensor, n_experts: int, ff: int, shared_ff: int,
-                         extra_cols: int = 0) -> torch.Tensor:
+                         extra_cols: int = 0, shared_gate: bool = True) -> torch.Tensor:
     """h[n, c] *= weight(n, expert of column c) in place, over the columns of all experts end to end (then a shared
-    expert's): for activations that a product's epilogue has gated already."""
+    expert's, which stay as they are without ``shared_gate``): for activations that a product's epilogue has gated
+    already."""
     N, F = h.shape
     if F != n_experts * ff + shared_ff:
         raise KernelError(f"scale_expert_columns: {F} columns for {n_experts} experts of {ff} and a shared one of {shared_ff}")
     _check(_fn("core", "mv_scale_expert_columns")(
         _need(h, "gated activations"), _dt(h),
-        _need(dense, "route weights", torch.float32, (N, n_experts + (1 if shared_ff else 0) + extra_cols)),
-        N, int(n_experts), int(ff), int(shared_ff), int(extra_cols), _stream()), "mv_scale_expert_columns")
+        _need(dense, "route weights", torch.float32, (N, n_experts + (1 if shared_ff and shared_gate else 0) + extra_cols)),
+        N, int(n_experts), int(ff), int(shared_ff), int(extra_cols), int(bool(shared_gate)), _stream()), "mv_scale_expert_columns")
     account(2 * N * F * h.element_size())
     return h
 
@@ -874,14 +904,15 @@ def expert_sort(pick: torch.Tensor, n_experts: int, x: torch.Tensor, rank: torch
 
 
 def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_group: torch.Tensor, n: int, k: int, *,
-                    row_step: int = 0, k_step: int = 0, swiglu: bool = False, active_rows: Optional[int] = None) -> torch.Tensor:
+                    row_step: int = 0, k_step: int = 0, swiglu: bool = False, active_rows: Optional[int] = None,
+                    limits: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One product for many groups, on the tcgen05 tensor cores (bfloat16): the rows of ``x`` [tiles * 128, k] are
     sorted by group with every group's run padded to whole tiles (:func:`expert_sort`), ``tile_group`` names each
     tile's group (negative: nothing to do), and ``w`` holds the groups' [n, k] matrices one below the other
     (``row_step`` rows a group) or side by side along its columns (``k_step`` columns a group).  ``out``
     [tiles * 128, n] float32 or bfloat16, or with ``swiglu`` bfloat16 [tiles * 128, n / 2] from rows of ``w`` that
-    alternate in groups of 16 gate and 16 up rows.  ``active_rows``: rows that belong to a group, for the profile's
-    accounts."""
+    alternate in groups of 16 gate and 16 up rows (``limits`` [n + 1], the same for every group: the clamped
+    activation, see :func:`glu_limits`).  ``active_rows``: rows that belong to a group, for the profile's accounts."""
     M = x.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError(f"gemm_tc_grouped: operands must be bfloat16, got {x.dtype} and {w.dtype}")
@@ -892,14 +923,15 @@ def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_gr
     if swiglu:
         if n % 32:
             raise KernelError(f"gemm_tc_grouped: the SwiGLU epilogue needs rows in groups of 32, got {n}")
-        mode, ldo = 3, n // 2
+        mode, ldo = (3 if limits is None else 4), n // 2
         _need(out, "gemm out", torch.bfloat16, (M, n // 2))
     else:
         mode, ldo = (0 if out.dtype == torch.float32 else 1), n
         _need(out, "gemm out", None, (M, n))
         _dt(out)
     _check(_fn("bf16", "mv_gemm_tc_grouped")(
-        _need(x, "gemm x"), _need(w, "gemm w"), out.data_ptr(), mode, M, int(n), int(k), ldo, w.shape[0], w.shape[1],
+        _need(x, "gemm x"), _need(w, "gemm w"), _need(limits, "activation limits", torch.float32, (n + 1,), True),
+        out.data_ptr(), mode, M, int(n), int(k), ldo, w.shape[0], w.shape[1],
         _need(tile_group, "tile groups", torch.int32), int(row_step), int(k_step), _error_flag(x.device).data_ptr(),
         _stream()), "mv_gemm_tc_grouped")
     rows = M if active_rows is None else active_rows
@@ -1146,10 +1178,12 @@ def attention_sink_prefill(q: torch.Tensor, pool: torch.Tensor, page_size: int, 
 
 
 def embed_bigram(table: torch.Tensor, bigram: torch.Tensor, tokens, positions, seq_of, cu, slots, prev: torch.Tensor,
-                 out: torch.Tensor, kept: Optional[torch.Tensor], mul_prev: int, mul_cur: int) -> torch.Tensor:
+                 out: torch.Tensor, kept: Optional[torch.Tensor], mul_prev: int, mul_cur: int,
+                 rounded: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[n] = table[token] + bigram[r] in float32, r = (previous token * mul_prev + token * mul_cur) mod buckets with
     buckets = rows of ``bigram`` - 1, or the last row for a token at position 0.  ``prev`` int32 [slots]: the last
-    token of each sequence before this step; it is brought up to date.  ``kept``: a second copy of the rows, or None."""
+    token of each sequence before this step; it is brought up to date.  ``kept``: a second copy of the rows, or None;
+    ``rounded``: the rows in its own dtype, or None."""
     N = tokens.numel()
     V, H = table.shape
     if bigram.dim() != 2 or bigram.shape[1] != H or bigram.shape[0] < 2 or bigram.dtype != table.dtype:
@@ -1161,6 +1195,7 @@ def embed_bigram(table: torch.Tensor, bigram: torch.Tensor, tokens, positions, s
         _need(positions, "positions", torch.int32), _need(seq_of, "seq_of", torch.int32), _need(cu, "cu", torch.int32),
         _need(slots, "slots", torch.int32), _need(prev, "previous tokens", torch.int32),
         _need(out, "embedding out", torch.float32, (N, H)), _need(kept, "embedding copy", torch.float32, (N, H), True),
+        _need(rounded, "embedding rounded", None, (N, H), True), _dt(rounded) if rounded is not None else F32,
         N, H, bigram.shape[0] - 1, int(mul_prev), int(mul_cur), _stream()), "mv_embed_bigram")
     account(N * H * (2 * table.element_size() + (8 if kept is not None else 4)))
     return out
@@ -1189,16 +1224,22 @@ LATENT_MAX_ROT = 512
 
 def latent_prepare(proj: torch.Tensor, q0: int, c0: int, w_c: torch.Tensor, eps: float, inv_freq: Optional[torch.Tensor],
                    positions, seq_of, page_table, pool: torch.Tensor, page_size: int, qa: torch.Tensor, nh: int, dim: int,
-                   rot: int, rank: int, rot_dims: Optional[int] = None) -> None:
+                   rot: int, rank: int, rot_dims: Optional[int] = None, cq0: int = 0, w_q: Optional[torch.Tensor] = None,
+                   cq: Optional[torch.Tensor] = None) -> None:
     """From float32 rows of a fused projection (q at column ``q0``: per head [dim | rot]; the latent at column ``c0``:
     [rank | rot]): the latent's first ``rank`` numbers over their root mean square times ``w_c``, its last ``rot`` and
     every head's last ``rot`` of q rotated (their first ``rot_dims``, all by default: element i with i + rot_dims / 2,
     angle pos * inv_freq[i]; the others pass unchanged); the row [rank + rot]
     goes into the token's place of its page, the rotated parts of q into the last ``rot`` columns of ``qa``
-    [N, nh, rank + rot] (float32; None: the queries are prepared elsewhere)."""
+    [N, nh, rank + rot] (float32; None: the queries are prepared elsewhere, and ``q0`` is not looked at).  ``cq``
+    [N, q_rank] in the pool's dtype: the queries' own latent, from column ``cq0``, over its root mean square times
+    ``w_q``."""
     N = proj.shape[0]
+    if qa is None:
+        q0 = 0
     if (not proj.is_cuda or proj.dtype != torch.float32 or proj.dim() != 2 or proj.stride(1) != 1
-            or q0 < 0 or q0 + nh * (dim + rot) > proj.shape[1] or c0 < 0 or c0 + rank + rot > proj.shape[1]):
+            or q0 < 0 or (qa is not None and q0 + nh * (dim + rot) > proj.shape[1]) or c0 < 0
+            or c0 + rank + rot > proj.shape[1] or (cq is not None and (cq0 < 0 or cq0 + cq.shape[1] > proj.shape[1]))):
         raise KernelError(f"latent_prepare: projection {proj.dtype} {tuple(proj.shape)} does not hold q at {q0} and the "
                           f"latent at {c0} for {N} rows")
     rot_dims = rot if rot_dims is None else int(rot_dims)
@@ -1212,28 +1253,39 @@ def latent_prepare(proj: torch.Tensor, q0: int, c0: int, w_c: torch.Tensor, eps:
         float(eps), _need(inv_freq, "inv_freq", torch.float32, (rot_dims // 2,), rot_dims == 0),
         _need(positions, "positions", torch.int32), _need(seq_of, "seq_of", torch.int32),
         _need(page_table, "page table", torch.int32), page_table.shape[1], int(page_size), pool.data_ptr(), pool.stride(0),
-        _dt(pool), _need(qa, "absorbed q", torch.float32, (N, nh, rank + rot), True), N, nh, dim, rot, rank, rot_dims, _stream()),
-        "mv_latent_prepare")
-    account(N * (nh * rot * 8 + (rank + rot) * (4 + pool.element_size())))
+        _dt(pool), _need(qa, "absorbed q", torch.float32, (N, nh, rank + rot), True), N, nh, dim, rot, rank, rot_dims,
+        int(cq0), cq.shape[1] if cq is not None else 0,
+        _need(w_q, "query latent norm weight", torch.float32, (cq.shape[1],)) if cq is not None else None,
+        _need(cq, "query latent", pool.dtype, (N, None), True), _stream()), "mv_latent_prepare")
+    account(N * ((nh * rot * 8 if qa is not None else 0) + (rank + rot + (cq.shape[1] if cq is not None else 0)) * (4 + pool.element_size())))
 
 
 def head_product(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, nh: int, n_in: int, n_out: int, *,
-                 transposed: bool = False, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 transposed: bool = False, gate: Optional[torch.Tensor] = None, rot: int = 0, rot_dims: int = 0,
+                 inv_freq: Optional[torch.Tensor] = None, positions=None) -> torch.Tensor:
     """One small matrix per head: y[n, h, :n_out] = W_h x[n, h, :n_in] with ``w`` [nh * n_out, n_in], or with
     ``transposed`` W_h^T x with ``w`` [nh * n_in, n_out].  ``x`` float32 [N, nh, >= n_in] and ``y`` [N, nh, >= n_out]
     (float32 or the model's dtype) may be views with any row and head strides.  ``gate``: float32 logits
-    [N, nh * n_out] (a column slice is fine); the result is multiplied by sigmoid(gate)."""
+    [N, nh * n_out], or [N, nh] for one a head (a column slice is fine); the result is multiplied by sigmoid(gate).
+    ``rot`` > 0: the ``rot`` elements of x after its ``n_in`` are turned (their first ``rot_dims``: i with
+    i + rot_dims / 2, angle positions * inv_freq[i]; the others pass unchanged) and written after y's ``n_out``
+    (float32)."""
     N = x.shape[0]
-    for t, what, width in ((x, "input", n_in), (y, "output", n_out)):
+    if rot and (y.dtype != torch.float32 or rot_dims % 2 or not 0 <= rot_dims <= rot):
+        raise KernelError(f"head_product: {rot_dims} of {rot} elements turned, output {y.dtype}")
+    for t, what, width in ((x, "input", n_in + rot), (y, "output", n_out + rot)):
         if not t.is_cuda or t.dim() != 3 or t.shape[0] != N or t.shape[1] != nh or t.shape[2] < width or t.stride(2) != 1:
             raise KernelError(f"head_product: {what} {tuple(t.shape)} strides {t.stride()} for {N} rows, {nh} heads of {width}")
     if x.dtype != torch.float32:
         raise KernelError(f"head_product: input is {x.dtype}, expected float32")
     rows, cols = (nh * n_in, n_out) if transposed else (nh * n_out, n_in)
-    gp, ldg = _cols(gate, "head_product gate", N, nh * n_out) if gate is not None else (None, 0)
+    per_head = gate is not None and gate.shape[1] == nh and n_out != 1
+    gp, ldg = _cols(gate, "head_product gate", N, nh if per_head else nh * n_out) if gate is not None else (None, 0)
     _check(_fn("core", "mv_head_product")(
         x.data_ptr(), x.stride(0), x.stride(1), _need(w, "head matrices", None, (rows, cols)), _dt(w), int(bool(transposed)),
-        gp, ldg, y.data_ptr(), _dt(y), y.stride(0), y.stride(1), N, nh, int(n_in), int(n_out), _stream()), "mv_head_product")
+        gp, ldg, int(per_head), y.data_ptr(), _dt(y), y.stride(0), y.stride(1), N, nh, int(n_in), int(n_out), int(rot),
+        int(rot_dims), _need(inv_freq, "inv_freq", torch.float32, (rot_dims // 2,)) if rot_dims else None,
+        _need(positions, "positions", torch.int32) if rot else None, _stream()), "mv_head_product")
     account(w.numel() * w.element_size() + N * nh * (n_in * 4 + n_out * y.element_size()), 2 * N * nh * n_in * n_out)
     return y
 
@@ -1328,17 +1380,19 @@ def latent_attention_prefill(q: torch.Tensor, kx: torch.Tensor, v0: int, r: torc
     """Causal softmax attention on the tensor cores for steps of many tokens: ``q`` [N, nh, dim + rot] against the
     gathered rows' keys and values ``kx`` [rows, >= v0 + nh dv] (head h's unrotated key at column h dim, its value at
     v0 + h dv) and the shared rotated key part ``r`` [rows, rot]; all bfloat16, scores and softmax float32.
-    ``gate``: float32 logits [N, nh dv] (a column slice is fine); ``out`` [N, nh dv] is multiplied by their sigmoid."""
+    ``gate``: float32 logits [N, nh dv], or [N, nh] for one a head (a column slice is fine); ``out`` [N, nh dv] is
+    multiplied by their sigmoid."""
     N, rows = q.shape[0], kx.shape[0]
     if not latent_prefill_fits(dim, rot, dv, 8):
         raise KernelError(f"latent_attention_prefill: sizes {dim} + {rot}, {dv} are not served")
     if kx.dtype != torch.bfloat16 or kx.dim() != 2 or kx.stride(1) != 1 or kx.shape[1] < v0 + nh * dv or v0 < nh * dim:
         raise KernelError(f"latent_attention_prefill: keys and values {kx.dtype} {tuple(kx.shape)}, values from {v0}")
-    gp, ldg = _cols(gate, "latent_attention_prefill gate", N, nh * dv) if gate is not None else (None, 0)
+    per_head = gate is not None and gate.shape[1] == nh
+    gp, ldg = _cols(gate, "latent_attention_prefill gate", N, nh if per_head else nh * dv) if gate is not None else (None, 0)
     _check(_fn("bf16", "mv_latent_attention_prefill")(
         _need(q, "q", torch.bfloat16, (N, nh, dim + rot)), kx.data_ptr(), kx.stride(0), int(v0),
         _need(r, "rotated keys", torch.bfloat16, (rows, rot)), _need(cu, "cu", torch.int32),
-        _need(starts, "starts", torch.int32), _need(sinks, "sinks", torch.float32, (nh,), True), gp, ldg,
+        _need(starts, "starts", torch.int32), _need(sinks, "sinks", torch.float32, (nh,), True), gp, ldg, int(per_head),
         _need(out, "attention out", torch.bfloat16, (N, nh * dv)), N, int(n_seqs), nh, dim, rot, dv, float(scale),
         int(window), _stream()), "mv_latent_attention_prefill")
     return out
@@ -1467,13 +1521,31 @@ class NormLink:
     n_partials: int = 0            # set by the emitting product
 
 
+def glu_limits(widths_and_limits, alpha: float, device) -> torch.Tensor:
+    """What the products' epilogues take to apply the clamped gated activation (:func:`glu_clamped`) to gate and up
+    rows that alternate in groups of 16: a limit a row of the matrix, then alpha.  ``widths_and_limits``: (features,
+    limit) of each run of features in the matrix's order."""
+    rows = [torch.full((2 * int(w),), float(limit), dtype=torch.float32) for w, limit in widths_and_limits]
+    return torch.cat(rows + [torch.tensor([float(alpha)], dtype=torch.float32)]).to(device)
+
+
+def _glu_mode(N: int, bias: Optional[torch.Tensor], limits: Optional[torch.Tensor]):
+    """(mode, row stride of the output, what goes in the bias's place) of a product whose epilogue gates."""
+    if limits is None:
+        return 3, N // 2, bias
+    if bias is not None:
+        raise KernelError("gemm: the clamped activation's epilogue takes no bias")
+    return 4, N // 2, limits
+
+
 def gemm_small_m_tile_rows(N: int, mode: int) -> int:
     return int(_fn("bf16", "mv_gemm_small_m_tile_rows")(int(N), int(mode)))
 
 
 def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
                  accumulate: bool = False, swiglu: bool = False, scale: Optional[NormLink] = None,
-                 emit: Optional[NormLink] = None, ahead: Optional[tuple] = None) -> torch.Tensor:
+                 emit: Optional[NormLink] = None, ahead: Optional[tuple] = None,
+                 limits: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out = x @ w.T for at most 64 rows of x, bfloat16 operands: the
     weight-streaming tensor-core kernel of the decode step.  ``scale`` / ``emit``: the
     two ends of a :class:`NormLink`.  ``ahead``: (address, bytes) of what the step's next
@@ -1490,7 +1562,7 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: O
     if swiglu:
         if N % 32:
             raise KernelError(f"gemm_small_m: the SwiGLU epilogue needs rows in groups of 32, got {N}")
-        mode, ldo = 3, N // 2
+        mode, ldo, bias = _glu_mode(N, bias, limits)
         _need(out, "gemm out", torch.bfloat16, (M, N // 2))
     elif accumulate:
         mode = 2
@@ -1501,7 +1573,7 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: O
         _dt(out)
     link = _link_args(x, M, N, K, mode, scale, emit, -(-N // gemm_small_m_tile_rows(N, 2)))
     _check(_fn("bf16", "mv_gemm_small_m")(
-        _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N,), True),
+        _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N + (mode == 4),), True),
         out.data_ptr(), mode, M, N, K, ldo, *link, *(ahead or (None, 0)), _stream()), "mv_gemm_small_m")
     _account_gemm(x, w, out, accumulate)
     return out
@@ -1699,7 +1771,8 @@ def gemm_tc_pair_takes(M: int, N: int) -> bool:
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
             accumulate: bool = False, swiglu: bool = False, pair: Optional[bool] = None,
-            scale: Optional[NormLink] = None, emit: Optional[NormLink] = None) -> torch.Tensor:
+            scale: Optional[NormLink] = None, emit: Optional[NormLink] = None,
+            limits: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out = x @ w.T, bfloat16 operands, on the tcgen05 tensor cores (TMA
     loads, accumulator in tensor memory): the matrix product of prefill.
     ``pair``: True: the kernel in which two multiprocessors share a 256 x 256 tile, False: the
@@ -1718,7 +1791,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
     if swiglu:
         if N % 32:
             raise KernelError(f"gemm_tc: the SwiGLU epilogue needs rows in groups of 32, got {N}")
-        mode, ldo = 3, N // 2
+        mode, ldo, bias = _glu_mode(N, bias, limits)
         _need(out, "gemm out", torch.bfloat16, (M, N // 2))
     elif accumulate:
         mode = 2
@@ -1736,7 +1809,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
             raise KernelError(f"gemm_tc: a product that emits a norm needs N in steps of 32, got {N}")
         link = _link_args(x, M, N, K, mode, scale, emit, -(-N // 256))
         _check(_fn("bf16", "mv_gemm_tc_pair")(
-            _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N,), True),
+            _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N + (mode == 4),), True),
             out.data_ptr(), mode, M, N, K, ldo, *link, _error_flag(x.device).data_ptr(), _stream()), "mv_gemm_tc_pair")
         _account_gemm(x, w, out, accumulate)
         return out
@@ -1745,7 +1818,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
     link = _link_args(x, M, N, K, mode, scale, None, 0)
     entry = "mv_gemm_tc"
     _check(_fn("bf16", entry)(
-        _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N,), True),
+        _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N + (mode == 4),), True),
         out.data_ptr(), mode, M, N, K, ldo, *link[:5], _error_flag(x.device).data_ptr(), _stream()), entry)
     _account_gemm(x, w, out, accumulate)
     return out
@@ -1753,7 +1826,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
 
 def gemm_tc_swap(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
                  accumulate: bool = False, swiglu: bool = False, scale: Optional[NormLink] = None,
-                 emit: Optional[NormLink] = None, ahead: Optional[tuple] = None) -> torch.Tensor:
+                 emit: Optional[NormLink] = None, ahead: Optional[tuple] = None,
+                 limits: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out = x @ w.T on the tcgen05 tensor cores with the operands' roles swapped (rows of w
     on the MMA's M side, up to 256 tokens a tile on its N side): a TMA pipeline that streams w
     once, K cut over the blocks of a cluster.  Same contract as ``gemm_small_m``, for any number of
@@ -1770,7 +1844,7 @@ def gemm_tc_swap(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: O
     if swiglu:
         if N % 32:
             raise KernelError(f"gemm_tc_swap: the SwiGLU epilogue needs rows in groups of 32, got {N}")
-        mode, ldo = 3, N // 2
+        mode, ldo, bias = _glu_mode(N, bias, limits)
         _need(out, "gemm out", torch.bfloat16, (M, N // 2))
     elif accumulate:
         mode = 2
@@ -1781,7 +1855,7 @@ def gemm_tc_swap(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: O
         _dt(out)
     link = _link_args(x, M, N, K, mode, scale, emit, -(-N // 128))
     _check(_fn("bf16", "mv_gemm_tc_swap")(
-        _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N,), True),
+        _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N + (mode == 4),), True),
         out.data_ptr(), mode, M, N, K, ldo, *link, *(ahead or (None, 0)), _error_flag(x.device).data_ptr(), _stream()),
         "mv_gemm_tc_swap")
     _account_gemm(x, w, out, accumulate)

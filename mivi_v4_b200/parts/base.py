@@ -44,6 +44,12 @@ class Part:
         A mixer or feed-forward that answers (False, False), the default, is never passed either."""
         return False, False
 
+    def take_side_rows(self, w) -> bool:
+        """Offer further rows (a matrix [n, hidden] that reads the same input) to the product that this part's forward
+        begins with.  A part that takes them (True; called once, after its tensors are loaded) leaves the rows' results,
+        float32 [N, n], in ``self.side`` after every forward; the default is not to."""
+        return False
+
     def scratch(self, step, name: str, shape, dtype):
         """A buffer from the step's workspace under a name of this part's kind: parts of different kinds
         never share one, so a part may hold its buffers across a call into another part.  (Layers of the

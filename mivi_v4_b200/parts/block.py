@@ -5,6 +5,7 @@ import torch
 
 from ..ops import kernels as K
 from ..ops.kernels import profile_stage
+from ..ops.linear import linear
 from .base import Part
 from .norm import LayerNorm, RMSNorm
 from .registry import register
@@ -318,6 +319,107 @@ class PostNormBlock(Part):
                 want = narrow and isinstance(after, PostNormBlock)
                 self._add(branches, self.ffn_norm, resid, rounded if want else None)
         if narrow and isinstance(after, PostNormBlock):
+            step.handed = ("stream", rounded)
+
+
+@register("block", "sum_norm")
+class SumNormBlock(Part):
+    """x <- norm1(alpha x + mixer(x)); then, if the layer has a feed-forward, x <- norm2(alpha x + feed_forward(x)): the
+    norms sit BEHIND the residual sum, so the stream itself is normed, and ``alpha`` weighs what it held (the arrangement
+    of DeepNet).  With ``gated`` a sublayer's result is multiplied element by element by sigmoid(W x + b) before the sum
+    (``rg1``, ``rg1.b`` the mixer's, ``rg2``, ``rg2.b`` the feed-forward's).  The norms are root-mean-square norms.  The
+    sublayers read the stream itself (rounded to the model's dtype where that is narrower) and write into a float32 buffer
+    of their own; ONE kernel per sublayer applies the gate, forms the sum, norms it into the float32 stream and writes the
+    rounded rows that the next sublayer multiplies.  A sublayer that begins with a product over float32 results
+    takes the gate's matrix along in it (``take_side_rows``)."""
+
+    nested_roles = {"mixer": "mixer", "mixer_norm": "norm", "ffn": "feed_forward", "ffn_norm": "norm"}
+
+    def __init__(self, hidden: int, alpha: float, mixer, mixer_norm, ffn=None, ffn_norm=None, gated: bool = False):
+        if (ffn is None) != (ffn_norm is None):
+            raise ValueError("a feed-forward and its norm come together or not at all")
+        for norm in (mixer_norm, ffn_norm):
+            if norm is not None and not isinstance(norm, RMSNorm):
+                raise ValueError("the norms of a sum_norm block are rmsnorm parts")
+        for part in (mixer, ffn):
+            if part is not None and not (getattr(part, "overwrites", False) or hasattr(part, "forward_sum")):
+                raise ValueError(f"{getattr(part, 'kind', '?')} cannot write its result apart from the residual stream")
+        self.hidden, self.alpha, self.gated = int(hidden), float(alpha), bool(gated)
+        self.mixer, self.mixer_norm, self.ffn, self.ffn_norm = mixer, mixer_norm, ffn, ffn_norm
+
+    def nested(self):
+        parts = {"mixer": self.mixer, "mixer_norm": self.mixer_norm, "ffn": self.ffn, "ffn_norm": self.ffn_norm}
+        return {k: v for k, v in parts.items() if v is not None}
+
+    def param_specs(self):
+        from .spec import ParamSpec
+        H = self.hidden
+        names = (["rg1"] + (["rg2"] if self.ffn is not None else [])) if self.gated else []
+        specs = {n: ParamSpec((H, H)) for n in names}
+        specs.update({n + ".b": ParamSpec((H,), "vector", "bias") for n in names})
+        return specs
+
+    def load_named(self, named) -> None:
+        super().load_named(named)                     # the sublayers' own tensors first: they may take the gate's rows
+        self.gate1, self.gate2 = getattr(self, "rg1", None), getattr(self, "rg2", None)
+        self.bias1, self.bias2 = getattr(self, "rg1_b", None), getattr(self, "rg2_b", None)
+        self.rg1 = self.rg2 = None
+        if self.gate1 is not None and self.mixer.take_side_rows(self.gate1):
+            self.gate1 = None
+        if self.gate2 is not None and self.ffn.take_side_rows(self.gate2):
+            self.gate2 = None
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def entry_link(self, step):
+        """No product carries this block's norms; the method is there so that the model tells ``forward`` which
+        block runs next (``after``)."""
+        return None
+
+    def _sublayer(self, part, norm, gate_w, gate_b, u, resid, rounded, step, *args) -> None:
+        N = u.shape[0]
+        with profile_stage(("mixer " if part is self.mixer else "feed_forward ") + getattr(part, "kind", "?")):
+            if hasattr(part, "forward_sum"):
+                branches = part.forward_sum(u, step, *args)
+            else:
+                y = self.scratch(step, "y", (N, self.hidden), torch.float32)
+                part.forward(u, y, step, *args, accumulate=False)
+                branches = [(y, 1.0)]
+        z = None
+        if self.gated:
+            if gate_w is None:
+                z = part.side
+            else:
+                z = self.scratch(step, "gate", (N, self.hidden), torch.float32)
+                with profile_stage("residual gate"):
+                    linear(u, gate_w, z)
+        (y1, s1), rest = branches[0], branches[1:]
+        if len(rest) > 1:
+            raise ValueError("at most two branches are summed in the norm's kernel")
+        y2, s2 = rest[0] if rest else (None, 1.0)
+        with profile_stage("norm"):
+            K.sum_norm(y1, resid, self.alpha, norm.weight, norm.eps, s1=s1, y2=y2, s2=s2, gate=z, gate_bias=gate_b, rounded=rounded)
+
+    def forward(self, resid, step, view, after=None) -> None:
+        N, H = resid.shape
+        narrow = step.dtype != torch.float32
+        handed, step.handed = getattr(step, "handed", None), None
+        rounded = step.ws.get("stream_rounded", (N, H), step.dtype) if narrow else None
+        if not narrow:
+            u = resid                                   # the sublayers multiply the stream itself
+        elif handed is not None and handed[0] == "stream":
+            u = handed[1]
+        else:
+            u = K.round_rows(resid, rounded)
+        # the rounded rows are wanted by this block's feed-forward, or by the next block of this kind
+        hand_on = narrow and isinstance(after, SumNormBlock)
+        want = rounded if narrow and (self.ffn is not None or hand_on) else None
+        self._sublayer(self.mixer, self.mixer_norm, self.gate1, self.bias1, u, resid, want, step, view)
+        if self.ffn is not None:
+            self._sublayer(self.ffn, self.ffn_norm, self.gate2, self.bias2, rounded if narrow else resid, resid,
+                           rounded if hand_on else None, step)
+        if hand_on:
             step.handed = ("stream", rounded)
 
 

@@ -75,13 +75,16 @@ class BigramEmbedding(Part):
     """x_t = E[token_t] + B[r_t]: a token embedding plus a row of a hashed bigram table,
     r_t = (token_(t-1) * mul_prev + token_t * mul_cur) mod buckets, and row ``buckets`` (the table's last) for a
     sequence's first token.  The previous token is part of a sequence's state: one int32 per slot.  With ``keep``
-    a second copy of the rows is left in ``step.embedding_output`` for parts that add it to the stream again later."""
+    a second copy of the rows is left in ``step.embedding_output`` for parts that add it to the stream again later; with
+    ``hand_rounded`` the rows are also handed to the first block in the model's dtype, as ("stream", rows) in ``step.handed``."""
 
-    def __init__(self, vocab: int, hidden: int, buckets: int, mul_prev: int, mul_cur: int, keep: bool = False):
+    def __init__(self, vocab: int, hidden: int, buckets: int, mul_prev: int, mul_cur: int, keep: bool = False,
+                 hand_rounded: bool = False):
         if buckets < 1:
             raise ValueError(f"a bigram table needs at least one bucket, got {buckets}")
         self.vocab, self.hidden, self.buckets = int(vocab), int(hidden), int(buckets)
         self.mul_prev, self.mul_cur, self.keep = int(mul_prev), int(mul_cur), bool(keep)
+        self.hand_rounded = bool(hand_rounded)
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         return {"weight": ParamSpec((self.vocab, self.hidden)), "bigram": ParamSpec((self.buckets + 1, self.hidden))}
@@ -98,9 +101,14 @@ class BigramEmbedding(Part):
         N = step.n_tokens
         x = step.ws.get("resid", (N, self.hidden), torch.float32)
         kept = step.ws.get("embedding_output", (N, self.hidden), torch.float32) if self.keep else None
+        rounded = None
+        if self.hand_rounded and step.dtype != torch.float32:
+            rounded = step.ws.get("stream_rounded", (N, self.hidden), step.dtype)
         K.embed_bigram(self.weight, self.bigram, step.tokens, step.positions, step.seq_of, step.cu, step.slots,
-                       view.state.view(-1), x, kept, self.mul_prev, self.mul_cur)
+                       view.state.view(-1), x, kept, self.mul_prev, self.mul_cur, rounded=rounded)
         step.embedding_output = kept
+        if self.hand_rounded:
+            step.handed = ("stream", rounded) if rounded is not None else None
         return x
 
 

@@ -93,16 +93,19 @@ class ClampedGLU(Part):
 
 @register("feed_forward", "routed_experts")
 class RoutedExperts(Part):
-    """Mixture of experts: every expert is W_down (silu(W_gate h) * (W_up h)) without
-    biases; router logits z = W_router h in float32, scores s = sigmoid(z), or with ``score`` "softmax" softmax(z)
-    over all routed entries; with ``correction`` a learned number per entry is added to the scores for the CHOICE
+    """Mixture of experts: every expert is W_down act(W_gate h, W_up h) without
+    biases, act = silu(g) * u, or with ``act`` "clamped" the clamped gated activation of ``clamped_glu`` (``limit``,
+    ``shared_limit`` for the shared expert, ``alpha``); router logits z = W_router h in float32 (with ``router_bias`` plus
+    a number an entry), scores s = sigmoid(z), or with ``score`` "softmax" softmax(z)
+    over all routed entries, or with "chosen_softmax" z itself, the weights then being softmax over the chosen z alone;
+    with ``correction`` a learned number per entry is added to the scores for the CHOICE
     only (the weights use the scores themselves); the weights are multiplied by ``out_scale``; the last
     ``n_identity`` routed entries (after the ``n_experts`` experts with matrices) are identity experts whose output
     is the input itself times the weight.  The entries form ``n_groups`` equal
     groups of neighbours, a group's score is the sum of its two largest scores, and only experts of the
     ``keep_groups`` best groups can be chosen; the ``top`` largest scores among them are chosen and weigh their
     experts by s / (sum of the chosen s + 1e-20).  With ``shared_ff`` > 0 a shared expert of that width runs for
-    every token and is added times sigmoid(w_sg . h).
+    every token and is added times sigmoid(w_sg . h), or as it is without ``shared_gate``.
 
     All experts' gate and up matrices are laid end to end (the shared expert's last), so that one product yields
     every expert's pre-activations; the gated activation is multiplied by the router's weight before it is
@@ -113,11 +116,12 @@ class RoutedExperts(Part):
 
     overwrites = True
 
-    SCORES = {"sigmoid": K.ROUTE_SIGMOID, "softmax": K.ROUTE_SOFTMAX}
+    SCORES = {"sigmoid": K.ROUTE_SIGMOID, "softmax": K.ROUTE_SOFTMAX, "chosen_softmax": K.ROUTE_CHOSEN_SOFTMAX}
 
     def __init__(self, hidden: int, n_experts: int, ff: int, top: int, n_groups: int = 1, keep_groups: int = 1,
                  shared_ff: int = 0, score: str = "sigmoid", correction: bool = False, out_scale: float = 1.0,
-                 n_identity: int = 0):
+                 n_identity: int = 0, router_bias: bool = False, shared_gate: bool = True, act: str = "silu",
+                 limit: float = 0.0, shared_limit: float = 0.0, alpha: float = 1.702):
         routed = int(n_experts) + int(n_identity)
         if n_experts < 1 or n_identity < 0 or routed > K.MAX_EXPERTS or n_groups < 1 or routed % n_groups:
             raise ValueError(f"{routed} routed entries do not form {n_groups} equal groups (at most {K.MAX_EXPERTS})")
@@ -126,28 +130,36 @@ class RoutedExperts(Part):
                              f"{routed // n_groups} (at most 32)")
         if score not in self.SCORES:
             raise ValueError(f"router score {score!r}; known: {', '.join(sorted(self.SCORES))}")
+        if act not in ("silu", "clamped") or (act == "clamped" and not (limit > 0 and (shared_limit > 0 or not shared_ff))):
+            raise ValueError(f"expert activation {act!r} with limits {limit} and {shared_limit}; known: silu, clamped (limits > 0)")
         self.hidden, self.E, self.ff, self.top = int(hidden), int(n_experts), int(ff), int(top)
         self.n_groups, self.keep, self.shared_ff = int(n_groups), int(keep_groups), int(shared_ff)
         self.score, self.has_correction, self.out_scale = score, bool(correction), float(out_scale)
         self.I, self.routed = int(n_identity), routed
+        self.has_router_bias, self.shared_gate = bool(router_bias), bool(shared_gate) and self.shared_ff > 0
+        self.clamped, self.limit, self.shared_limit, self.alpha = act == "clamped", float(limit), float(shared_limit), float(alpha)
+        self.side, self._side_at = None, None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         H, F = self.hidden, self.ff
         specs = {"router": ParamSpec((self.routed, H))}
         if self.has_correction:
             specs["correction"] = ParamSpec((self.routed,), "vector", "bias")
+        if self.has_router_bias:
+            specs["router.b"] = ParamSpec((self.routed,), "vector", "bias")
         for e in range(self.E):
             specs.update({f"e{e}.gate": ParamSpec((F, H)), f"e{e}.up": ParamSpec((F, H)), f"e{e}.down": ParamSpec((H, F))})
         if self.shared_ff:
             S = self.shared_ff
-            specs.update({"shared.gate": ParamSpec((S, H)), "shared.up": ParamSpec((S, H)), "shared.down": ParamSpec((H, S)),
-                          "shared.sg": ParamSpec((1, H))})
+            specs.update({"shared.gate": ParamSpec((S, H)), "shared.up": ParamSpec((S, H)), "shared.down": ParamSpec((H, S))})
+            if self.shared_gate:
+                specs["shared.sg"] = ParamSpec((1, H))
         return specs
 
     def active_matrix_elements(self) -> int:
         """Matrix elements that one token is multiplied with: the router, its chosen experts, the shared one."""
         H = self.hidden
-        return self.routed * H + 3 * self.top * self.ff * H + (3 * self.shared_ff * H + H if self.shared_ff else 0)
+        return self.routed * H + 3 * self.top * self.ff * H + 3 * self.shared_ff * H + (H if self.shared_gate else 0)
 
     def load(self, t) -> None:
         names = [f"e{e}." for e in range(self.E)] + (["shared."] if self.shared_ff else [])
@@ -168,15 +180,29 @@ class RoutedExperts(Part):
         self.shared_group = G if self.shared_ff and self.shared_ff % G == 0 else 0
         self.w_gu = torch.cat([gate_up(n, self.shared_ff if n == "shared." else self.ff) for n in names], dim=0).contiguous()
         self.w_down = torch.cat([t[n + "down"] for n in names], dim=1).contiguous()
-        rows = [t["router"]] + ([t["shared.sg"]] if self.shared_ff else [])
+        rows = [t["router"]] + ([t["shared.sg"]] if self.shared_gate else [])
         pad = -sum(r.shape[0] for r in rows) % 16
         if pad:
             rows.append(torch.zeros((pad, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
         self.w_router = torch.cat(rows, dim=0).contiguous()
-        self.correction = t.get("correction")
+        self.correction, self.router_bias = t.get("correction"), t.get("router.b")
+        # the clamped activation inside the products: a limit a row of the gate and up matrices (one expert's; all)
+        self.expert_limits = self.all_limits = self.shared_limits = None
+        if self.clamped:
+            device = self.w_gu.device
+            self.expert_limits = K.glu_limits([(self.ff, self.limit)], self.alpha, device)
+            self.shared_limits = K.glu_limits([(self.shared_ff, self.shared_limit)], self.alpha, device)
+            self.all_limits = K.glu_limits([(self.E * self.ff, self.limit), (self.shared_ff, self.shared_limit)], self.alpha, device)
         # the shared expert's down matrix by itself, for the steps that sort the tokens by expert (kept in a list,
         # beside the weights that every step reads: a copy of columns that those steps read from it instead)
         self._shared_down = [self.w_down[:, self.E * self.ff:].contiguous()] if self.shared_ff else []
+
+    def take_side_rows(self, w) -> bool:
+        if w.dtype != self.w_router.dtype:
+            return False
+        self._side_at = (self.w_router.shape[0], w.shape[0])
+        self.w_router = torch.cat([self.w_router, w]).contiguous()
+        return True
 
     # Steps that bring an expert this many rows on average (never a decode step) sort the (token, choice) entries
     # by expert and run ONE grouped product over the sorted rows for the experts' gate and up matrices and one for
@@ -199,27 +225,32 @@ class RoutedExperts(Part):
     def forward(self, g, resid, step, accumulate: bool = True) -> None:
         N = g.shape[0]
         E, F, I = self.E, self.E * self.ff + self.shared_ff, self.I
-        sg = 1 if self.shared_ff else 0
+        sg = 1 if self.shared_gate else 0
         cols = self.routed + sg                  # a dense row: [experts | the shared gate | identity experts]
         z = self.scratch(step, "z", (N, self.w_router.shape[0]), torch.float32)
         linear(g, self.w_router, z)
+        if self._side_at is not None:
+            self.side = z[:, self._side_at[0]:self._side_at[0] + self._side_at[1]]
         dense = self.scratch(step, "route", (N, cols), torch.float32)
         pick = self.scratch(step, "pick", (N, self.top), torch.int32)
         pick_w = self.scratch(step, "pick_w", (N, self.top), torch.float32)
-        K.route(z[:, :cols], dense, pick, pick_w, self.routed, self.n_groups, self.keep, self.top, bool(self.shared_ff),
-                mode=self.SCORES[self.score], correction=self.correction, out_scale=self.out_scale, n_identity=I)
+        K.route(z[:, :cols], dense, pick, pick_w, self.routed, self.n_groups, self.keep, self.top, self.shared_gate,
+                mode=self.SCORES[self.score], correction=self.correction, out_scale=self.out_scale, n_identity=I,
+                bias=self.router_bias)
         if self._sorted_ok(g, step, N):
             return self._forward_sorted(g, resid, step, accumulate, dense, pick, pick_w)
         h = self.scratch(step, "ffh", (N, F), step.dtype)
         if (N >= self.GATED_IN_PRODUCT_FROM and self.group and (self.shared_group or not self.shared_ff)
                 and tensor_core_ok(g, self.w_gu)):
             # long steps: gate and up never reach memory; the weights go on the rounded activations
-            linear_swiglu(g, self.w_gu, h)
-            K.scale_expert_columns(h, dense, E, self.ff, self.shared_ff, extra_cols=I)
+            linear_swiglu(g, self.w_gu, h, limits=self.all_limits)
+            K.scale_expert_columns(h, dense, E, self.ff, self.shared_ff, extra_cols=I, shared_gate=self.shared_gate)
         else:
             gu = self.scratch(step, "proj", (N, 2 * F), torch.float32)
             linear(g, self.w_gu, gu)
-            K.routed_glu(gu, dense, h, E, self.ff, self.shared_ff, self.group, self.shared_group, extra_cols=I)
+            clamp = dict(limit=self.limit, shared_limit=self.shared_limit, alpha=self.alpha) if self.clamped else {}
+            K.routed_glu(gu, dense, h, E, self.ff, self.shared_ff, self.group, self.shared_group, extra_cols=I,
+                         shared_gate=self.shared_gate, **clamp)
         linear(h, self.w_down, resid, accumulate=accumulate)
         if I:
             K.identity_experts(g, dense, E + sg, I, resid)
@@ -237,7 +268,8 @@ class RoutedExperts(Part):
         xs = self.scratch(step, "sorted", (rows, H), g.dtype)
         K.expert_sort(pick, E, g, rank, counts, place, xs, offsets, tile_group)
         hs = self.scratch(step, "sorted_h", (rows, ff), step.dtype)
-        K.gemm_tc_grouped(xs, self.w_gu, hs, tile_group, 2 * ff, H, row_step=2 * ff, swiglu=True, active_rows=N * top)
+        K.gemm_tc_grouped(xs, self.w_gu, hs, tile_group, 2 * ff, H, row_step=2 * ff, swiglu=True, active_rows=N * top,
+                          limits=self.expert_limits)
         ys = self.scratch(step, "sorted_y", (rows, H), torch.float32)
         K.gemm_tc_grouped(hs, self.w_down, ys, tile_group, H, ff, k_step=ff, active_rows=N * top)
         shared = None
@@ -245,12 +277,15 @@ class RoutedExperts(Part):
             hsh = self.scratch(step, "shared_h", (N, self.shared_ff), step.dtype)
             w_gu = self.w_gu[E * 2 * ff:]
             if self.shared_group and tensor_core_ok(g, w_gu):
-                linear_swiglu(g, w_gu, hsh)
+                linear_swiglu(g, w_gu, hsh, limits=self.shared_limits)
             else:
                 gu = self.scratch(step, "proj", (N, w_gu.shape[0]), torch.float32)
                 linear(g, w_gu, gu)
-                K.swiglu(gu, hsh, self.shared_group)
+                if self.clamped:
+                    K.glu_clamped(gu, hsh, self.shared_limit, self.alpha, self.shared_group)
+                else:
+                    K.swiglu(gu, hsh, self.shared_group)
             shared = self.scratch(step, "shared_y", (N, H), torch.float32)
             linear(hsh, self._shared_down[0], shared)
-        # the shared expert's gate is the last column of the router's dense weights
-        K.expert_combine(ys, place, pick_w, shared, dense[:, E:E + 1] if shared is not None else None, resid, accumulate)
+        # the shared expert's gate, where it has one, is the last column of the router's dense weights
+        K.expert_combine(ys, place, pick_w, shared, dense[:, E:E + 1] if self.shared_gate else None, resid, accumulate)

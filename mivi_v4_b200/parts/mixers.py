@@ -651,7 +651,9 @@ class LatentAttention(Part):
     square and multiplied by a weight (the latent c), and ``rot_dim`` more, one rotated key part r shared by all
     heads; per head the unrotated key is W_uk c and the value W_uv c; score = (q_unrotated . k_unrotated +
     q_rotated . r) * scale; a sliding ``window`` (0: none); with ``sink`` a learned number per head joins the softmax's
-    denominator; with ``gated`` the concatenated heads are multiplied by sigmoid(W_g h); then W_o.  The position
+    denominator; with ``gated`` the concatenated heads are multiplied by sigmoid(W_g h), element by element ("element",
+    or True) or head by head ("head": W_g has a row a head); then W_o.  With ``q_rank`` the queries come through a latent
+    of their own: q = W_uq c_q, c_q = W_dq h over its root mean square times a weight.  The position
     part turns the first ``position.head_dim`` of the ``rot_dim`` elements, element i with i + head_dim / 2.
 
     Only [c | r] is cached, one row a token for all heads.  W_uk is folded into the query
@@ -662,12 +664,16 @@ class LatentAttention(Part):
     overwrites = True
 
     def __init__(self, hidden: int, n_heads: int, dim: int, rot_dim: int, value_dim: int, kv_rank: int, scale: float,
-                 eps: float, position, window: int = 0, sink: bool = True, gated: bool = True):
+                 eps: float, position, window: int = 0, sink: bool = True, gated=True, q_rank: int = 0):
+        if gated not in (True, False, "element", "head"):
+            raise ValueError(f"output gate {gated!r}; known: element, head, or none")
         if not 1 <= kv_rank <= K.LATENT_MAX_RANK or not 0 <= rot_dim <= K.LATENT_MAX_ROT:
             raise ValueError(f"latent size {kv_rank} (1..{K.LATENT_MAX_RANK}), rotated size {rot_dim} (0..{K.LATENT_MAX_ROT})")
         self.hidden, self.nh, self.dim, self.rd = int(hidden), int(n_heads), int(dim), int(rot_dim)
         self.dv, self.rank, self.scale, self.eps = int(value_dim), int(kv_rank), float(scale), float(eps)
         self.window, self.sink, self.gated, self.position = int(window), bool(sink), bool(gated), position
+        self.gate_rows = 0 if not gated else (self.nh if gated == "head" else self.nh * self.dv)
+        self.q_rank = int(q_rank)
         self.rot_dims = 0
         if isinstance(position, Rope):
             if position.style != "half_split" or position.head_dim > self.rd:
@@ -681,23 +687,34 @@ class LatentAttention(Part):
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         H, nh, qd, dv, rank = self.hidden, self.nh, self.dim + self.rd, self.dv, self.rank
-        specs = {"q": ParamSpec((nh * qd, H)), "dkv": ParamSpec((rank + self.rd, H)),
-                 "dkv.norm": ParamSpec((rank,), "vector", "norm"), "uk": ParamSpec((nh * self.dim, rank)),
-                 "uv": ParamSpec((nh * dv, rank)), "o": ParamSpec((H, nh * dv))}
+        if self.q_rank:
+            specs = {"dq": ParamSpec((self.q_rank, H)), "dq.norm": ParamSpec((self.q_rank,), "vector", "norm"),
+                     "uq": ParamSpec((nh * qd, self.q_rank))}
+        else:
+            specs = {"q": ParamSpec((nh * qd, H))}
+        specs.update({"dkv": ParamSpec((rank + self.rd, H)), "dkv.norm": ParamSpec((rank,), "vector", "norm"),
+                      "uk": ParamSpec((nh * self.dim, rank)), "uv": ParamSpec((nh * dv, rank)), "o": ParamSpec((H, nh * dv))})
         if self.sink:
             specs["sink"] = ParamSpec((nh,), "vector", "bias")
         if self.gated:
-            specs["g"] = ParamSpec((nh * dv, H))
+            specs["g"] = ParamSpec((self.gate_rows, H))
         return specs
 
     def load(self, t) -> None:
-        self.w_in = _fuse_rows([t["q"], t["dkv"]] + ([t["g"]] if self.gated else []))
+        self.w_in = _fuse_rows([t["dq" if self.q_rank else "q"], t["dkv"]] + ([t["g"]] if self.gated else []))
         self.c_norm, self.sinks, self.w_o = t["dkv.norm"], t.get("sink"), t["o"]
-        self.w_uk, self.w_uv = t["uk"].contiguous(), t["uv"].contiguous()
+        self.q_norm, self.w_uq = t.get("dq.norm"), t.get("uq")
+        self.w_kv = _fuse_rows([t["uk"], t["uv"]])            # keys' and values' matrices of all heads, one above the other
         # steps of many tokens build every head's keys and values from the cached rows with one product
-        self.w_kv = None
-        if self.w_uk.dtype == torch.bfloat16 and K.latent_prefill_fits(self.dim, self.rd, self.dv, self.rank):
-            self.w_kv = _fuse_rows([self.w_uk, self.w_uv])
+        self.long_ok = self.w_kv.dtype == torch.bfloat16 and K.latent_prefill_fits(self.dim, self.rd, self.dv, self.rank)
+        self.side, self._side_at = None, None
+
+    def take_side_rows(self, w) -> bool:
+        if w.dtype != self.w_in.dtype:
+            return False
+        self._side_at = (self.w_in.shape[0], w.shape[0])
+        self.w_in = torch.cat([self.w_in, w]).contiguous()
+        return True
 
     def cache_need(self):
         return KVNeed(1, self.rank + self.rd, self.window, self.rank, values_in_keys=True)
@@ -713,25 +730,39 @@ class LatentAttention(Part):
     def forward(self, u, resid, step, view, accumulate: bool = True) -> None:
         N = u.shape[0]
         nh, dim, rd, dv, rank = self.nh, self.dim, self.rd, self.dv, self.rank
-        c0 = nh * (dim + rd)
+        c0 = self.q_rank or nh * (dim + rd)
         g0 = c0 + rank + rd
+        w_uk, w_uv = self.w_kv[:nh * dim], self.w_kv[nh * dim:nh * (dim + dv)]
         proj = self.scratch(step, "proj", (N, self.w_in.shape[0]), torch.float32)
         linear(u, self.w_in, proj)
+        if self._side_at is not None:
+            self.side = proj[:, self._side_at[0]:self._side_at[0] + self._side_at[1]]
         rot = self.position.rotary(u.device) if self.rot_dims else None
         inv_freq = rot[0] if rot is not None else None
-        gate = proj[:, g0:g0 + nh * dv] if self.gated else None
+        gate = proj[:, g0:g0 + self.gate_rows] if self.gated else None
         y = self.scratch(step, "mix", (N, nh * dv), step.dtype)
         rows = self._seen_rows(step) if step.max_len >= self.LONG_STEP else 0
         if K.profiling_on():
             reach = self.window or None
             pairs = sum(sum(min(s + i + 1, reach) if reach else s + i + 1 for i in range(n))
                         for s, n in zip(step.host_starts, step.host_lens))
-        if (self.w_kv is not None and step.dtype == torch.bfloat16 and view.pool.dtype == torch.bfloat16
-                and 0 < rows <= self.LONG_ROWS * N):
-            K.latent_prepare(proj, 0, c0, self.c_norm, self.eps, inv_freq, step.positions, step.seq_of, view.page_table,
-                             view.pool, view.page_size, None, nh, dim, rd, rank, self.rot_dims)
+        long = (self.long_ok and step.dtype == torch.bfloat16 and view.pool.dtype == torch.bfloat16
+                and 0 < rows <= self.LONG_ROWS * N)
+        queries, cq, qa = proj, None, None
+        if self.q_rank:
+            # the queries come out of a second product, which reads the normed latent
+            cq = self.scratch(step, "cq", (N, self.q_rank), step.dtype)
+            queries = self.scratch(step, "queries", (N, nh * (dim + rd)), torch.float32)
+        if not long:
+            qa = self.scratch(step, "qa", (N, nh, rank + rd), torch.float32)
+        K.latent_prepare(proj, 0, c0, self.c_norm, self.eps, inv_freq, step.positions, step.seq_of, view.page_table,
+                         view.pool, view.page_size, None if self.q_rank else qa, nh, dim, rd, rank, self.rot_dims,
+                         w_q=self.q_norm, cq=cq)
+        if self.q_rank:
+            linear(cq, self.w_uq, queries)
+        if long:
             q = self.scratch(step, "q", (N, nh, dim + rd), torch.bfloat16)
-            K.latent_query(proj, 0, inv_freq, step.positions, q, nh, dim, rd, self.rot_dims)
+            K.latent_query(queries, 0, inv_freq, step.positions, q, nh, dim, rd, self.rot_dims)
             c = self.scratch(step, "c", (rows, rank), torch.bfloat16)
             r = self.scratch(step, "r", (rows, rd), torch.bfloat16)
             K.latent_gather(view.pool, view.page_size, view.page_table, step.cu, step.starts, step.n_seqs, self.window, c, r)
@@ -744,10 +775,9 @@ class LatentAttention(Part):
                           2 * nh * (dim + rd + 2 * dv) * pairs)
             linear(y, self.w_o, resid, accumulate=accumulate)
             return
-        qa = self.scratch(step, "qa", (N, nh, rank + rd), torch.float32)
-        K.latent_prepare(proj, 0, c0, self.c_norm, self.eps, inv_freq, step.positions, step.seq_of, view.page_table,
-                         view.pool, view.page_size, qa, nh, dim, rd, rank, self.rot_dims)
-        K.head_product(proj[:, :c0].unflatten(1, (nh, dim + rd)), self.w_uk, qa, nh, dim, rank, transposed=True)
+        # (queries that latent_prepare did not see are turned here)
+        turn = dict(rot=rd, rot_dims=self.rot_dims, inv_freq=inv_freq, positions=step.positions) if self.q_rank and rd else {}
+        K.head_product(queries[:, :nh * (dim + rd)].unflatten(1, (nh, dim + rd)), w_uk, qa, nh, dim, rank, transposed=True, **turn)
         o_lat = self.scratch(step, "o_lat", (N, nh, rank), torch.float32)
         # few query tokens with many keys each: the keys in shares.  The number of shares follows from what the page
         # table can hold, not from the lengths of the moment, so that a recorded step stays right as they grow.
@@ -762,7 +792,7 @@ class LatentAttention(Part):
         if K.profiling_on():
             K.account((rank + rd) * view.pool.element_size() * pairs + N * nh * (2 * rank + rd) * 4,
                       2 * nh * (2 * rank + rd) * pairs)
-        K.head_product(o_lat, self.w_uv, y.view(N, nh, dv), nh, rank, dv, gate=gate)
+        K.head_product(o_lat, w_uv, y.view(N, nh, dv), nh, rank, dv, gate=gate)
         linear(y, self.w_o, resid, accumulate=accumulate)
 
 

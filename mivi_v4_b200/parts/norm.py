@@ -15,17 +15,20 @@ from .spec import ParamSpec
 class RMSNorm(Part):
     """y = x * (mean(x^2) + eps)^-1/2 * weight over the last dimension, in
     float32 (crates/mivi-core/src/simd/norm.rs:38-72; math.rs:14-29).  ``one_plus``: the checkpoint stores the
-    weight around zero and the factor is 1 + weight (added once, in float32, when the weights are loaded)."""
+    weight around zero and the factor is 1 + weight (added once, in float32, when the weights are loaded).  ``scalar``: the
+    checkpoint stores ONE number for all coordinates (a tensor without dimensions), spread over them when the weights are
+    loaded."""
 
-    def __init__(self, dim: int, eps: float, one_plus: bool = False):
-        self.dim, self.eps, self.one_plus = int(dim), float(eps), bool(one_plus)
+    def __init__(self, dim: int, eps: float, one_plus: bool = False, scalar: bool = False):
+        self.dim, self.eps, self.one_plus, self.scalar = int(dim), float(eps), bool(one_plus), bool(scalar)
         self.weight: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {"weight": ParamSpec((self.dim,), "vector", "bias" if self.one_plus else "norm")}
+        return {"weight": ParamSpec(() if self.scalar else (self.dim,), "vector", "bias" if self.one_plus else "norm")}
 
     def load(self, t) -> None:
-        self.weight = (t["weight"].float() + 1.0).contiguous() if self.one_plus else t["weight"]
+        w = t["weight"].float() + 1.0 if self.one_plus else t["weight"]
+        self.weight = (w.expand(self.dim) if self.scalar else w).contiguous()
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         return K.rmsnorm(x, self.weight, self.eps, out, rows)
