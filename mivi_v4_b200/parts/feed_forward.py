@@ -220,7 +220,7 @@ class RoutedExperts(Part):
     def _sorted_ok(self, g, step, N: int) -> bool:
         return (N * self.top >= self.SORTED_ROWS_AN_EXPERT * self.E and not step.is_decode and self.top < self.E
                 and self.I == 0 and self.group == K.SWIGLU_GROUP and self.ff % 8 == 0 and g.shape[1] % 8 == 0
-                and tensor_core_ok(g, self.w_gu) and self.w_down.dtype == torch.bfloat16)
+                and tensor_core_ok(g, self.w_gu) and self.w_down.dtype == torch.bfloat16 and self.w_down.shape[1] % 8 == 0)
 
     def forward(self, g, resid, step, accumulate: bool = True) -> None:
         N = g.shape[0]
