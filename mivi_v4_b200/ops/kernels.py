@@ -115,6 +115,7 @@ _SIGNATURES = {
                                       _I, _I, _P, _P, _I, _I, _P, _I, _P],
         "mv_attention_decode_tc": [_P, _P, _Q, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _P, _P],
         "mv_attention_prefill_tc": [_P, _P, _Q, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
+        "mv_latent_attention_decode": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P, _P],
         "mv_latent_query": [_P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "mv_latent_gather": [_P, _Q, _P, _I, _I, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P],
         "mv_latent_attention_prefill": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P],
@@ -1330,6 +1331,48 @@ def latent_attention(qa: torch.Tensor, pool: torch.Tensor, page_size: int, page_
         _need(part[0], "shares", torch.float32, (N, nh, splits, rank)) if splits > 1 else None,
         _need(part[1], "shares' sums", torch.float32, (N, nh, splits, 2)) if splits > 1 else None,
         _stream()), "mv_latent_attention")
+    return out
+
+
+LATENT_DECODE_KEYS, LATENT_DECODE_HEADS, LATENT_DECODE_COLS, LATENT_DECODE_MAX_WIDTH = 64, 16, 256, 680
+
+
+def latent_decode_fits(dtype: torch.dtype, rank: int, rot: int) -> bool:
+    """Whether the tensor-core kernel for steps of few tokens takes a cache of this dtype and these sizes."""
+    return dtype == torch.bfloat16 and rank % 8 == 0 and rot % 8 == 0 and -(-(rank + rot) // 16) * 16 <= LATENT_DECODE_MAX_WIDTH
+
+
+def latent_decode_splits(n_tokens: int, n_heads: int, rank: int, longest: int, sm_count: int) -> int:
+    """Into how many shares of the keys :func:`latent_attention_decode` cuts a step of ``n_tokens`` query tokens: two
+    blocks a multiprocessor, no share under a tile of keys."""
+    blocks = max(1, n_tokens * -(-n_heads // LATENT_DECODE_HEADS) * -(-rank // LATENT_DECODE_COLS))
+    return int(max(1, min(2 * sm_count // blocks, longest // LATENT_DECODE_KEYS, LATENT_MAX_SPLITS)))
+
+
+def latent_attention_decode(qa: torch.Tensor, pool: torch.Tensor, page_size: int, page_table, positions, seq_of,
+                            out: torch.Tensor, nh: int, rank: int, rot: int, scale: float, *, window: int = 0,
+                            sinks: Optional[torch.Tensor] = None, splits: int = 1,
+                            part: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> torch.Tensor:
+    """:func:`latent_attention` on the tensor cores, for a bfloat16 cache (``latent_decode_fits``): 16 heads a block are
+    the rows of both products; queries and softmax weights enter them as two bfloat16 numbers each (16 bits of
+    mantissa)."""
+    N = qa.shape[0]
+    if not latent_decode_fits(pool.dtype, rank, rot):
+        raise KernelError(f"latent_attention_decode: a {pool.dtype} cache of rows of {rank} + {rot} is not served")
+    _check_latent_pool(pool, page_size, rank + rot, "latent_attention_decode")
+    splits = int(splits)
+    if not 1 <= splits <= LATENT_MAX_SPLITS or (splits > 1 and part is None):
+        raise KernelError(f"latent_attention_decode: {splits} shares of the keys (1..{LATENT_MAX_SPLITS}) need their scratch")
+    _guard("bf16", "latent_attention_decode", qa.device, n_pages=pool.shape[0])
+    _check(_fn("bf16", "mv_latent_attention_decode")(
+        _need(qa, "absorbed q", torch.float32, (N, nh, rank + rot)), pool.data_ptr(), pool.stride(0),
+        _need(page_table, "page table", torch.int32), page_table.shape[1], int(page_size),
+        _need(positions, "positions", torch.int32), _need(seq_of, "seq_of", torch.int32),
+        _need(sinks, "sinks", torch.float32, (nh,), True), _need(out, "attention out", torch.float32, (N, nh, rank)),
+        N, nh, rank, rot, float(scale), int(window), splits,
+        _need(part[0], "shares", torch.float32, (N, nh, splits, rank)) if splits > 1 else None,
+        _need(part[1], "shares' sums", torch.float32, (N, nh, splits, 2)) if splits > 1 else None,
+        _error_flag(qa.device).data_ptr(), _stream()), "mv_latent_attention_decode")
     return out
 
 

@@ -782,13 +782,17 @@ class LatentAttention(Part):
         # few query tokens with many keys each: the keys in shares.  The number of shares follows from what the page
         # table can hold, not from the lengths of the moment, so that a recorded step stays right as they grow.
         longest = view.page_table.shape[1] * view.page_size
-        splits = K.latent_splits(N, nh, min(longest, self.window) if self.window else longest, K.n_sms())
+        longest = min(longest, self.window) if self.window else longest
+        if K.latent_decode_fits(view.pool.dtype, rank, rd):
+            attend, splits = K.latent_attention_decode, K.latent_decode_splits(N, nh, rank, longest, K.n_sms())
+        else:
+            attend, splits = K.latent_attention, K.latent_splits(N, nh, longest, K.n_sms())
         part = None
         if splits > 1:
             part = (self.scratch(step, "part_o", (N, nh, splits, rank), torch.float32),
                     self.scratch(step, "part_ml", (N, nh, splits, 2), torch.float32))
-        K.latent_attention(qa, view.pool, view.page_size, view.page_table, step.positions, step.seq_of, o_lat, nh, rank,
-                           rd, self.scale, window=self.window, sinks=self.sinks, splits=splits, part=part)
+        attend(qa, view.pool, view.page_size, view.page_table, step.positions, step.seq_of, o_lat, nh, rank, rd, self.scale,
+               window=self.window, sinks=self.sinks, splits=splits, part=part)
         if K.profiling_on():
             K.account((rank + rd) * view.pool.element_size() * pairs + N * nh * (2 * rank + rd) * 4,
                       2 * nh * (2 * rank + rd) * pairs)

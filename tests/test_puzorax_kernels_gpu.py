@@ -150,7 +150,8 @@ def _latent_case(T, H, dim, rd, vd, rank, window, rot_dims, base, scale, seed, l
     return h, p, m, P.latent_attention(h, p, m, 1e-5)
 
 
-def _run_latent(k, dtype, h, p, m, cuts, page_size, sink=True, splits=1):
+def _run_latent(k, dtype, h, p, m, cuts, page_size, sink=True, splits=1, tensor=False):
+    """``tensor``: the kernel for steps of few tokens that runs on the tensor cores."""
     from mivi_v4_b200.parts.position import Rope
     T = h.shape[0]
     H, dim, rd, vd, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
@@ -172,13 +173,18 @@ def _run_latent(k, dtype, h, p, m, cuts, page_size, sink=True, splits=1):
         k.head_product(proj[rows][:, :c0].unflatten(1, (H, dim + rd)), dev(p["uk"], dtype), qa, H, dim, rank, transposed=True)
         o_lat = torch.full((n, H, rank), float("nan"), device=DEV)
         part = (torch.full((n, H, splits, rank), float("nan"), device=DEV), torch.full((n, H, splits, 2), float("nan"), device=DEV))
-        k.latent_attention(qa, pool, page_size, table, pos, seq_of, o_lat, H, rank, rd, m["scale"], window=window,
-                           sinks=dev(p["sink"]) if sink else None, splits=splits, part=part if splits > 1 else None)
+        attend = k.latent_attention_decode if tensor else k.latent_attention
+        attend(qa, pool, page_size, table, pos, seq_of, o_lat, H, rank, rd, m["scale"], window=window,
+               sinks=dev(p["sink"]) if sink else None, splits=splits, part=part if splits > 1 else None)
         y = torch.full((n, H * vd), float("nan"), dtype=dtype, device=DEV)
         k.head_product(o_lat, dev(p["uv"], dtype), y.view(n, H, vd), H, rank, vd, gate=proj[rows][:, g0:g0 + H * vd])
         outs.append(y)
         at += n
     return torch.cat(outs)
+
+
+def _kernels(k, dtype, rank, rd):
+    return (False, True) if k.latent_decode_fits(dtype, rank, rd) else (False,)
 
 
 LATENT_SIZES = [(10, 8, 12, 6, 24, 10, 8, 100.0, 8), (1, 20, 0, 20, 36, 0, 0, 1.0, 16), (3, 4, 6, 10, 40, 70, 6, 1e4, 8),
@@ -192,7 +198,8 @@ def test_latent_attention_under_every_cut(dtype, H, dim, rd, vd, rank, window, r
     h, p, m, want = _latent_case(T, H, dim, rd, vd, rank, window, rot_dims, base, 0.3, seed=rank)
     tol = 3e-5 if dtype == torch.float32 else 2e-2
     for cuts in ([T], [1] * T, [100] + [1] * 70, [7] * 24 + [2], [63, 65, 42]):
-        close(_run_latent(k, dtype, h, p, m, cuts, page), want, tol, f"cuts {cuts[:3]}")
+        for tensor in _kernels(k, dtype, rank, rd):
+            close(_run_latent(k, dtype, h, p, m, cuts, page, tensor=tensor), want, tol, f"cuts {cuts[:3]}, tensor cores {tensor}")
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -206,7 +213,9 @@ def test_a_loud_key_far_away_and_just_inside_and_just_outside_a_window(dtype):
                               (64, 76, True), (64, 75, False), (1, 139, True), (1, 138, False)):
         h, p, m, want = _latent_case(T, H, dim, rd, vd, rank, window, 16, 1e6, 0.5, seed=key + window, loud=(139, key))
         for cuts in ([T], [120] + [1] * 20, [139, 1]):
-            close(_run_latent(k, dtype, h, p, m, cuts, 16), want, tol, f"window {window} loud key {key} cuts {cuts[:2]}")
+            for tensor in _kernels(k, dtype, rank, rd):
+                close(_run_latent(k, dtype, h, p, m, cuts, 16, tensor=tensor), want, tol,
+                      f"window {window} loud key {key} cuts {cuts[:2]}, tensor cores {tensor}")
         # the loud key decides the row where it is seen: the test would notice a mask that is one off
         c = P.rms_norm(h[key:key + 1, H * (dim + rd):H * (dim + rd) + rank], p["dkv.norm"], 1e-5)
         v_key = (c @ p["uv"].T)[0] * torch.sigmoid(h[139, H * (dim + rd) + rank + rd:])
@@ -224,9 +233,12 @@ def test_keys_in_shares_give_the_same_attention(dtype, splits):
     for T, window in ((170, 0), (170, 70), (40, 0), (3, 0)):
         h, p, m, want = _latent_case(T, 3, 8, 8, 8, 24, window, 8, 1e4, 0.4, seed=T + window)
         for cuts in ([T], [T - 2, 1, 1]):
-            close(_run_latent(k, dtype, h, p, m, cuts, 16, splits=splits), want, tol, f"{splits} shares, window {window}")
-        close(_run_latent(k, dtype, h, p, dict(m), [T], 16, sink=False, splits=splits),
-              P.latent_attention(h, dict(p, sink=torch.full((3,), -800.0, dtype=F64)), m, 1e-5), tol, "no sink")
+            for tensor in _kernels(k, dtype, 24, 8):
+                close(_run_latent(k, dtype, h, p, m, cuts, 16, splits=splits, tensor=tensor), want, tol,
+                      f"{splits} shares, window {window}, tensor cores {tensor}")
+        for tensor in _kernels(k, dtype, 24, 8):
+            close(_run_latent(k, dtype, h, p, dict(m), [T], 16, sink=False, splits=splits, tensor=tensor),
+                  P.latent_attention(h, dict(p, sink=torch.full((3,), -800.0, dtype=F64)), m, 1e-5), tol, "no sink")
 
 
 def test_number_of_shares_follows_the_work():
@@ -235,6 +247,9 @@ def test_number_of_shares_follows_the_work():
     assert k.latent_splits(8, 32, 100, 148) == 1                     # nothing to cut
     assert 2 <= k.latent_splits(8, 32, 4096, 148) <= k.LATENT_MAX_SPLITS
     assert k.latent_splits(1, 8, 1 << 20, 148) == k.LATENT_MAX_SPLITS
+    assert k.latent_decode_splits(2048, 32, 256, 4096, 148) == 1 and k.latent_decode_splits(8, 32, 256, 100, 148) == 1
+    assert k.latent_decode_splits(64, 32, 256, 4096, 148) == 2 and k.latent_decode_splits(8, 32, 256, 1 << 20, 148) == 18
+    assert k.latent_decode_splits(64, 32, 512, 4096, 148) == 1 and k.latent_decode_splits(1, 8, 64, 1 << 20, 148) == k.LATENT_MAX_SPLITS
 
 
 def _run_latent_long(k, h_seqs, p, m, steps, page_size):

@@ -174,6 +174,7 @@ def _run(part, h_seqs, steps, dtype, page=16, splits=None, monkeypatch=None):
     k = K()
     if splits is not None:
         monkeypatch.setattr(k, "latent_splits", lambda *a: splits)
+        monkeypatch.setattr(k, "latent_decode_splits", lambda *a: splits)
     per = [-(-x.shape[0] // page) for x in h_seqs]
     perm = torch.randperm(sum(per) + 3, generator=torch.Generator().manual_seed(5))[:sum(per)].tolist()      # pages in no order
     rows, at = [], 0
