@@ -116,6 +116,7 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1
 // size), gridDim.y = row tiles.
 // TAIL 1 (RT == 3): the three row tiles of a warp are N rows apart, N counts channels, see ConvTail.
 // TAIL 2 (RT == 4): a tile is one head, see HeadTail.
+// TAIL 3 (RT == 2): mode 4, the clamped gated activation.
 template <int NT, int RT, int UNROLL, int WARPS, int TAIL>
 __global__ void __launch_bounds__(WARPS * 32)
 gemm_small_m_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __restrict__ X,
@@ -430,13 +431,13 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __
             ss = mv_warp_sum(ss);
             v *= 1.0f / sqrtf(ss * link.inv_dim + link.eps);
         }
-        if (bias && mode != 4 && r < ROWS && n < N) v += bias[n];
-        if (mode >= 3) {
+        if (TAIL != 3 && bias && r < ROWS && n < N) v += bias[n];
+        if (TAIL == 3 || mode == 3) {
             // ROWS == 32: lanes 0-15 hold gate rows, lanes 16-31 the up rows of the same features
             const float up = __shfl_down_sync(0xffffffffu, v, 16);
             if (lane < 16 && n + 16 < N)
                 ((__nv_bfloat16*)out)[(size_t)m * ldo + (n >> 5) * 16 + lane] =
-                    __float2bfloat16_rn(mode == 4 ? mv_glu_clamped(v, up, bias[n], bias[N]) : mv_glu_silu(v, up));
+                    __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v, up, bias[n], bias[N]) : mv_glu_silu(v, up));
         } else {
             float sq = 0.f;
             if (r < ROWS && n < N) {
@@ -551,7 +552,15 @@ MV_API int mv_gemm_small_m(const void* X, const void* W, const float* bias, void
     }
     const int nt = (M + 7) / 8;
     const bool wide = mv_gemm_small_m_tile_rows(N, mode) == 32;
-#define MV_GO(NT, RT, U, WARPS) return launch<NT, RT, U, WARPS>(W, X, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, Ahead{next_w, next_bytes}, stream)
+#define MV_GO(NT, RT, U, WARPS)                                                                                                 \
+    do {                                                                                                                        \
+        if constexpr (RT == 2)                                                                                                  \
+            if (mode == 4)                                                                                                      \
+                return launch<NT, RT, U, WARPS, 3>(W, X, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{},            \
+                                                   Ahead{next_w, next_bytes}, stream);                                          \
+        return launch<NT, RT, U, WARPS>(W, X, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, Ahead{next_w, next_bytes}, \
+                                        stream);                                                                                \
+    } while (0)
     // few tokens: small blocks, many per SM; many tokens: large blocks, so that X is re-read less
     switch (nt) {
         case 1: if (wide) MV_GO(1, 2, 2, 4); else MV_GO(1, 1, 4, 4);

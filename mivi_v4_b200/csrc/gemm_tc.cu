@@ -64,7 +64,7 @@ struct SmemLayout {
     static constexpr int TOTAL = TILE_BYTES + BAR_BYTES + 1024;      // 1024 for the manual alignment
 };
 
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool CLAMP>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                const float* __restrict__ bias, void* __restrict__ out, int mode, int M, int N, int K, int ldo,
@@ -158,7 +158,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 tmem_ld32(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)c0, r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 if (rs.part) scale_chunk(r, sc);
-                if (row < M) store_chunk(r, row, n0 + c0, N, mode, bias, out, ldo);
+                if (row < M) store_chunk<CLAMP>(r, row, n0 + c0, N, mode, bias, out, ldo);
             }
         }
     }
@@ -190,7 +190,7 @@ struct WideLayout {
     static constexpr int TOTAL = TILE_BYTES + BAR_BYTES + 1024;
 };
 
-template <int STAGES>
+template <int STAGES, bool CLAMP>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     const float* __restrict__ bias, void* __restrict__ out, int mode, int M, int N, int K, int ldo,
@@ -299,7 +299,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 tmem_ld32(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)(acc * BN + c0), r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 if (rs.part) scale_chunk(r, sc);
-                if (row < M) store_chunk(r, row, n0 + c0, N, mode, bias, out, ldo);
+                if (row < M) store_chunk<CLAMP>(r, row, n0 + c0, N, mode, bias, out, ldo);
             }
             // this warp has read its lanes of the accumulator: hand it back
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -324,7 +324,7 @@ int sm_count() {
     return n;
 }
 
-template <int STAGES>
+template <int STAGES, bool CLAMP>
 int launch_wide(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
                 const RowScale& rs, int* err, cudaStream_t stream) {
     using L = WideLayout<STAGES>;
@@ -332,16 +332,16 @@ int launch_wide(const void* X, const void* W, const float* bias, void* out, int 
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, N, K, L::BN, &mb)) return (int)cudaErrorInvalidValue;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(gemm_tc_wide_kernel<STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_wide_kernel<STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         attr_set = true;
     }
     const int tiles = ((M + BM - 1) / BM) * ((N + L::BN - 1) / L::BN);
     const int blocks = tiles < sm_count() ? tiles : sm_count();
-    gemm_tc_wide_kernel<STAGES><<<blocks, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, err);
+    gemm_tc_wide_kernel<STAGES, CLAMP><<<blocks, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, err);
     return mv_launch_status();
 }
 
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool CLAMP>
 int launch(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
            const RowScale& rs, int* err, cudaStream_t stream) {
     using L = SmemLayout<BN, STAGES>;
@@ -349,16 +349,16 @@ int launch(const void* X, const void* W, const float* bias, void* out, int mode,
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, N, K, BN, &mb)) return (int)cudaErrorInvalidValue;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         attr_set = true;
     }
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
-    gemm_tc_kernel<BN, STAGES><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, err, nullptr, 0, 0);
+    gemm_tc_kernel<BN, STAGES, CLAMP><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, err, nullptr, 0, 0);
     return mv_launch_status();
 }
 
 // The grouped form: X [M, K] sorted by group, W [w_rows, w_cols] holding every group's matrix.
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool CLAMP>
 int launch_grouped(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo, int w_rows, int w_cols,
                    const int* tile_group, int b_row_step, int b_k_step, int* err, cudaStream_t stream) {
     using L = SmemLayout<BN, STAGES>;
@@ -366,11 +366,11 @@ int launch_grouped(const void* X, const void* W, const float* bias, void* out, i
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, w_rows, w_cols, BN, &mb)) return (int)cudaErrorInvalidValue;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         attr_set = true;
     }
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
-    gemm_tc_kernel<BN, STAGES><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, RowScale{}, err,
+    gemm_tc_kernel<BN, STAGES, CLAMP><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, RowScale{}, err,
                                                                    tile_group, b_row_step, b_k_step);
     return mv_launch_status();
 }
@@ -392,18 +392,21 @@ MV_API int mv_gemm_tc(const void* X, const void* W, const float* bias, void* out
     if (scale_part && (n_scale_part <= 0 || n_scale_part > scale_stride || dim <= 0)) return (int)cudaErrorInvalidValue;
     RowScale rs = {};
     if (scale_part) rs = RowScale{scale_part, n_scale_part, scale_stride, 1.0f / (float)dim, eps};
-    if (N <= 64) return launch<64, 4>(X, W, bias, out, mode, M, N, K, ldo, rs, err, stream);
+#define TC_GO(FN, ...) return mode == 4 ? FN<__VA_ARGS__, true>(X, W, bias, out, mode, M, N, K, ldo, rs, err, stream) \
+                                        : FN<__VA_ARGS__, false>(X, W, bias, out, mode, M, N, K, ldo, rs, err, stream)
+    if (N <= 64) TC_GO(launch, 64, 4);
     // wide enough for 128 x 256 tiles to give every SM work: the persistent kernel
     const long long wide_tiles = (long long)((M + BM - 1) / BM) * ((N + 255) / 256);
-    if (N >= 256 && wide_tiles >= 96) return launch_wide<4>(X, W, bias, out, mode, M, N, K, ldo, rs, err, stream);
-    return launch<128, 3>(X, W, bias, out, mode, M, N, K, ldo, rs, err, stream);
+    if (N >= 256 && wide_tiles >= 96) TC_GO(launch_wide, 4);
+    TC_GO(launch, 128, 3);
+#undef TC_GO
 }
 
 // The grouped product: the rows of X [M, K] are sorted by group and padded so that every tile of 128 rows belongs
 // to one group (tile_group [M / 128], negative for spare tiles); W [w_rows, w_cols] holds the groups' matrices one
 // below the other (b_row_step rows a group, b_k_step 0) or side by side along K (b_k_step columns a group, a
-// multiple of 8; b_row_step 0); N and K are ONE group's sizes.  Modes as mv_gemm_tc (no carried norm; bias, or mode 4's limits, are the
-// same for every group).
+// multiple of 8; b_row_step 0); N and K are ONE group's sizes.  Modes as mv_gemm_tc (no carried norm; bias, or mode 4's limits, are
+// the same for every group).
 // A tile's rows beyond its group's real rows hold whatever X holds there and give rows of ``out`` that nobody reads.
 MV_API int mv_gemm_tc_grouped(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
                               int w_rows, int w_cols, const int* tile_group, int b_row_step, int b_k_step, int* err,
@@ -412,7 +415,12 @@ MV_API int mv_gemm_tc_grouped(const void* X, const void* W, const float* bias, v
     if (K <= 0 || K % 8 || M % BM || b_k_step % 8 || !tile_group || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
         return (int)cudaErrorInvalidValue;
     if (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
-    if (N <= 64)
-        return launch_grouped<64, 4>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, b_k_step, err, stream);
-    return launch_grouped<128, 3>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, b_k_step, err, stream);
+#define TC_GO(BN, S)                                                                                                       \
+    return mode == 4 ? launch_grouped<BN, S, true>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, \
+                                                   b_k_step, err, stream)                                                  \
+                     : launch_grouped<BN, S, false>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, \
+                                                    b_k_step, err, stream)
+    if (N <= 64) TC_GO(64, 4);
+    TC_GO(128, 3);
+#undef TC_GO
 }

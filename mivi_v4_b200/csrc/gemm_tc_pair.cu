@@ -99,7 +99,7 @@ __device__ __forceinline__ void arrive_remote(unsigned cluster_addr) {
     asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(cluster_addr) : "memory");
 }
 
-template <int STAGES>
+template <int STAGES, bool CLAMP>
 __global__ void __launch_bounds__(PAIR_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     const float* __restrict__ bias, void* __restrict__ out, int mode, int M, int N, int K, int ldo,
@@ -305,7 +305,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                         for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
                     }
-                    if (row < M) store_chunk(r, row, n0 + c0, N, mode, bias, out, ldo);
+                    if (row < M) store_chunk<CLAMP>(r, row, n0 + c0, N, mode, bias, out, ldo);
                 }
             }
             // this warp has read its lanes of the accumulator: tell the leader's MMA warp
@@ -322,7 +322,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     }
 }
 
-template <int STAGES>
+template <int STAGES, bool CLAMP>
 int launch_pair(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
                 const PairLink& link, int* err, cudaStream_t stream) {
     using L = PairLayout<STAGES>;
@@ -330,7 +330,7 @@ int launch_pair(const void* X, const void* W, const float* bias, void* out, int 
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, N, K, PAIR_BN / 2, &mb)) return (int)cudaErrorInvalidValue;
     static int max_pairs = 0;
     if (max_pairs == 0) {
-        cudaFuncSetAttribute(gemm_tc_pair_kernel<STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_pair_kernel<STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         int dev = 0, sms = 148;
         cudaGetDevice(&dev);
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
@@ -345,7 +345,7 @@ int launch_pair(const void* X, const void* W, const float* bias, void* out, int 
         probe.attrs = pa;
         probe.numAttrs = 1;
         int n = 0;
-        if (cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel<STAGES>, &probe) != cudaSuccess || n <= 0) n = sms / 2;
+        if (cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel<STAGES, CLAMP>, &probe) != cudaSuccess || n <= 0) n = sms / 2;
         max_pairs = n < sms / 2 ? n : sms / 2;
         cudaGetLastError();
     }
@@ -363,7 +363,7 @@ int launch_pair(const void* X, const void* W, const float* bias, void* out, int 
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = mv_pdl_enabled() ? 2 : 1;
-    cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<STAGES>, ma, mb, bias, out, mode, M, N, K, ldo, link, err);
+    cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<STAGES, CLAMP>, ma, mb, bias, out, mode, M, N, K, ldo, link, err);
     return mv_launch_status();
 }
 
@@ -400,5 +400,6 @@ MV_API int mv_gemm_tc_pair(const void* X, const void* W, const float* bias, void
     }
     link.by_rows = (mode == 0 || mode == 2) && N % 32 == 0 && ldo % 4 == 0 && !(((uintptr_t)out | (uintptr_t)bias) & 15);
     if (emit_x && !link.by_rows) return (int)cudaErrorInvalidValue;
-    return launch_pair<6>(X, W, bias, out, mode, M, N, K, ldo, link, err, stream);
+    if (mode == 4) return launch_pair<6, true>(X, W, bias, out, mode, M, N, K, ldo, link, err, stream);
+    return launch_pair<6, false>(X, W, bias, out, mode, M, N, K, ldo, link, err, stream);
 }

@@ -4,26 +4,28 @@
 // such columns, ``bias`` then holding a limit a column and, after them, alpha).  Included inside the
 // including file's own namespace.
 // One row's 32 consecutive columns of the accumulator, from registers to Y, in the mode asked for.
+// CLAMP: mode 4, an instance of its own (the branch would cost the other modes registers).
+template <bool CLAMP>
 __device__ __forceinline__ void store_chunk(const unsigned (&r)[32], int row, int n_base, int N, int mode,
                                             const float* __restrict__ bias, void* __restrict__ out, int ldo) {
 
-        if (mode >= 3) {
+        if (CLAMP || mode == 3) {
             // columns n_base .. +15 are gate, +16 .. +31 the up values of the same features
             if (n_base + 32 <= N) {
                 __nv_bfloat16* dst = (__nv_bfloat16*)out + (size_t)row * ldo + (n_base >> 1);
                 unsigned packed[8];
-                const float limit = mode == 4 ? bias[n_base] : 0.f, alpha = mode == 4 ? bias[N] : 0.f;
+                const float limit = CLAMP ? bias[n_base] : 0.f, alpha = CLAMP ? bias[N] : 0.f;
 #pragma unroll
                 for (int j = 0; j < 16; j += 2) {
                     float a0 = __uint_as_float(r[j]), a1 = __uint_as_float(r[j + 1]);
                     float b0 = __uint_as_float(r[j + 16]), b1 = __uint_as_float(r[j + 17]);
-                    if (bias && mode == 3) {
+                    if (!CLAMP && bias) {
                         a0 += bias[n_base + j]; a1 += bias[n_base + j + 1];
                         b0 += bias[n_base + j + 16]; b1 += bias[n_base + j + 17];
                     }
                     const __nv_bfloat162 v =
-                        mode == 4 ? __floats2bfloat162_rn(mv_glu_clamped(a0, b0, limit, alpha), mv_glu_clamped(a1, b1, limit, alpha))
-                                  : __floats2bfloat162_rn(mv_glu_silu(a0, b0), mv_glu_silu(a1, b1));
+                        CLAMP ? __floats2bfloat162_rn(mv_glu_clamped(a0, b0, limit, alpha), mv_glu_clamped(a1, b1, limit, alpha))
+                              : __floats2bfloat162_rn(mv_glu_silu(a0, b0), mv_glu_silu(a1, b1));
                     packed[j >> 1] = *reinterpret_cast<const unsigned*>(&v);
                 }
                 if ((((uintptr_t)dst) & 15) == 0) {

@@ -372,12 +372,12 @@ gemm_tc_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                     for (int e = 0; e < 4; ++e) v[e] *= sc;
                 }
-                if (bias && mode != 4) {
+                if (TAIL != 3 && bias) {
 #pragma unroll
                     for (int e = 0; e < 4; ++e)
                         if (n + e < N) v[e] += bias[n + e];
                 }
-                if (mode >= 3) {
+                if (TAIL == 3 || mode == 3) {                // (TAIL 3: mode 4, the clamped gated activation)
                     // rows in groups of 16 gate + 16 up: of every 8 lanes the first 4 hold gate rows,
                     // the next 4 the up rows of the same features
                     float up[4];
@@ -387,7 +387,7 @@ gemm_tc_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         __nv_bfloat16* o = (__nv_bfloat16*)out + (size_t)m * ldo + (n >> 5) * 16 + (r & 15);
 #pragma unroll
                         for (int e = 0; e < 4; ++e)
-                            o[e] = __float2bfloat16_rn(mode == 4 ? mv_glu_clamped(v[e], up[e], bias[n], bias[N])
+                            o[e] = __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v[e], up[e], bias[n], bias[N])
                                                                  : mv_glu_silu(v[e], up[e]));
                     }
                 } else {
@@ -520,17 +520,20 @@ MV_API int mv_gemm_tc_swap(const void* X, const void* W, const float* bias, void
         // More tokens: tiles of 128 tokens along the grid's z (three stages of 32 KB, two blocks a
         // multiprocessor).  Tiles of 256 tokens (one block a multiprocessor) measured slower at every size:
         // each block reads its own copy of X from the L2 cache, and that traffic grows with the tile.
-        return launch<128, 3>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream,
-                              k_slices(N, K, 2, (M + 127) / 128));
+        const int slices = k_slices(N, K, 2, (M + 127) / 128);
+        if (mode == 4)
+            return launch<128, 3, 3>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices);
+        return launch<128, 3>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices);
     }
     const int slices = k_slices(N, K);
     const bool deep = slices == 1;
-#define MV_GO(BN) return deep ? launch<BN, 8>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices) \
-                              : launch<BN, 4>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices)
+#define MV_SWAP(BN, S, TAIL) launch<BN, S, TAIL>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices)
+#define MV_GO(BN) return mode == 4 ? (deep ? MV_SWAP(BN, 8, 3) : MV_SWAP(BN, 4, 3)) : (deep ? MV_SWAP(BN, 8, 0) : MV_SWAP(BN, 4, 0))
     if (M <= 16) MV_GO(16);
     if (M <= 32) MV_GO(32);
     MV_GO(64);
 #undef MV_GO
+#undef MV_SWAP
 }
 
 namespace {
