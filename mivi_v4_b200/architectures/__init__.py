@@ -1,2 +1,2 @@
 """One file per architecture; importing this package registers them all."""
-from . import lfm2, puzorax, redisun, ropelix, tevirax, votavik  # noqa: F401
+from . import lfm2, mevulix, puzorax, redisun, ropelix, tevirax, votavik  # noqa: F401

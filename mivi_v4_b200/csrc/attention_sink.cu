@@ -15,7 +15,11 @@
 //     by longer vectors);
 //   * a chunked mask: query i reads key j <= i only if both lie in the same chunk of `chunk` positions,
 //     counted from the sequence's position 0.
-//   * a distance bias: r1_h ln(1 + r2_h (i - j)) is taken off the score of query i and key j, two numbers a head;
+//   * a distance bias: r1_h ln(1 + r2_h (i - j)) is taken off the score of query i and key j, two numbers a head; or a
+//     learned number a head and distance, read from a table whose last column serves every longer distance.  Both
+//     come after the cap;
+//   * a factor on q that grows with the position p, 1 + coef ln(floor((p + 1) / every) + 1);
+//   * a layer that reads another layer's keys and values: q alone is prepared (nkv 0);
 //   * values that are the keys (the first dv elements of a key row): a page then holds key rows only;
 //   * a gate per token and ELEMENT of the concatenated heads instead of one per head;
 //   * every query head's weights applied to the values of EVERY kv head (32-bit results [token][head][kv head][dv]),
@@ -40,7 +44,7 @@ qkv_prepare_wide_kernel(const float* __restrict__ proj, int ld, const float* __r
                         const int* __restrict__ positions, const int* __restrict__ seq_of,
                         const int* __restrict__ page_table, int table_stride, int page_shift, T* __restrict__ pool,
                         long long page_stride, T* __restrict__ q_out, int nh, int nkv, int dk, int dv, int per_head,
-                        float amplitude) {
+                        float amplitude, float q_coef, float q_every) {
     mv_pdl_begin();
     extern __shared__ float head_scale[];           // [nh + nkv] with per_head
     __shared__ float scratch[33];
@@ -80,8 +84,9 @@ qkv_prepare_wide_kernel(const float* __restrict__ proj, int ld, const float* __r
     }
     __syncthreads();                                 // the rotation's table is complete whatever norm ran
     const int pos = positions[n];
+    const float q_mul = q_every > 0.f ? fmaf(q_coef, logf(floorf((float)(pos + 1) / q_every) + 1.0f), 1.0f) : 1.f;
     const int page_size = 1 << page_shift;
-    const int page = page_table[(size_t)seq_of[n] * table_stride + (pos >> page_shift)];
+    const int page = nkv > 0 ? page_table[(size_t)seq_of[n] * table_stride + (pos >> page_shift)] : 0;
     const int prow = pos & (page_size - 1);
     T* kpage = pool + (size_t)page * page_stride;
     T* vpage = kpage + (size_t)nkv * page_size * dk;
@@ -96,6 +101,7 @@ qkv_prepare_wide_kernel(const float* __restrict__ proj, int ld, const float* __r
         const float* w = is_q ? wq : wk;
         const int head = f / dk, d = f - head * dk;
         const float sc = per_head ? (w ? head_scale[is_q ? head : nh + head] : 1.f) : (is_q ? q_scale : k_scale);
+        const float mul = is_q ? q_mul : 1.f;
         const int wo = per_head ? head * dk : 0;           // a per-head weight is indexed inside the head
         float a = src[f] * sc * (w ? w[f - wo] : 1.f);
         if (d < rot_dims) {
@@ -107,7 +113,7 @@ qkv_prepare_wide_kernel(const float* __restrict__ proj, int ld, const float* __r
             a = d < half ? a * cs - b * sn : a * cs + b * sn;
         }
         if (is_q)
-            q_out[(size_t)n * nq + f] = mv_from_f32<T>(a);
+            q_out[(size_t)n * nq + f] = mv_from_f32<T>(a * mul);
         else if (page_ok)
             kpage[((size_t)head * page_size + prow) * dk + d] = mv_from_f32<T>(a);
     }
@@ -124,7 +130,7 @@ MV_API int mv_qkv_prepare_wide(const float* proj, int ld, const float* wq, const
                                const float* inv_freq, const int* positions, const int* seq_of, const int* page_table,
                                int table_stride, int page_size, void* pool, long long page_stride, void* q_out,
                                int dtype, int N, int nh, int nkv, int dk, int dv, int per_head, float amplitude,
-                               cudaStream_t stream) {
+                               float q_coef, float q_every, cudaStream_t stream) {
     if (N <= 0) return 0;
     const size_t smem = per_head ? sizeof(float) * (size_t)(nh + nkv) : 0;
     if ((page_size & (page_size - 1)) || rot_dims % 2 || rot_dims > dk || (rot_dims && !inv_freq) || smem > 32768)
@@ -137,11 +143,11 @@ MV_API int mv_qkv_prepare_wide(const float* proj, int ld, const float* wq, const
     if (dtype == MV_DT_BF16)
         mv_launch(qkv_prepare_wide_kernel<__nv_bfloat16>, grid, 256, smem, stream, proj, ld, wq, wk, eps, rot_dims, inv_freq,
                   positions, seq_of, page_table, table_stride, page_shift, (__nv_bfloat16*)pool, page_stride,
-                  (__nv_bfloat16*)q_out, nh, nkv, dk, dv, per_head, amplitude);
+                  (__nv_bfloat16*)q_out, nh, nkv, dk, dv, per_head, amplitude, q_coef, q_every);
     else
         mv_launch(qkv_prepare_wide_kernel<float>, grid, 256, smem, stream, proj, ld, wq, wk, eps, rot_dims, inv_freq,
                   positions, seq_of, page_table, table_stride, page_shift, (float*)pool, page_stride, (float*)q_out, nh,
-                  nkv, dk, dv, per_head, amplitude);
+                  nkv, dk, dv, per_head, amplitude, q_coef, q_every);
     return mv_launch_status();
 }
 
@@ -176,8 +182,8 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ pool, long 
                       const int* __restrict__ positions, const int* __restrict__ seq_of,
                       const float* __restrict__ sinks, const float* __restrict__ gate, int ld_gate,
                       T* __restrict__ o, int N, int nh, int nkv, int dk, int dv, float scale, float cap, int window,
-                      int keep_first, int chunk, const float* __restrict__ r1, const float* __restrict__ r2, int v_in_k,
-                      int gate_wide, float* __restrict__ o_all) {
+                      int keep_first, int chunk, const float* __restrict__ r1, const float* __restrict__ r2,
+                      const float* __restrict__ dist, int dist_len, int v_in_k, int gate_wide, float* __restrict__ o_all) {
     mv_pdl_begin();
     extern __shared__ __align__(16) float as_smem[];
     float* qs = as_smem;                            // [GT][dk]
@@ -263,7 +269,6 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ pool, long 
 #pragma unroll
             for (int i = 0; i < GT; ++i) {
                 s[i] = dot[i] * scale;
-                if (r1 && i < n_heads) s[i] -= r1[h0 + i] * log1pf(r2[h0 + i] * (float)(pos - t));
                 if (cap > 0.f) {
                     if (sizeof(T) == 2) {
                         // a bfloat16 run: tanh(x) = (1 - e^-2|x|) / (1 + e^-2|x|) with the fast exponential, as in the
@@ -274,6 +279,8 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ pool, long 
                         s[i] = cap * tanhf(s[i] * inv_cap);
                     }
                 }
+                if (r1 && i < n_heads) s[i] -= r1[h0 + i] * log1pf(r2[h0 + i] * (float)(pos - t));
+                if (dist && i < n_heads) s[i] += dist[(size_t)(h0 + i) * dist_len + min(pos - t, dist_len - 1)];
             }
         }
 #pragma unroll
@@ -369,17 +376,18 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ pool, long 
 }
 
 // head_tile: see below.  q [N, nh * dk]; o [N, nh * dv]; sinks [nh] or null; gate: 32-bit logits, gate[n * ld_gate + h]
-// (with gate_wide gate[n * ld_gate + h * dv + d]), or null; r1, r2 [nh] or null; v_in_k: the values are the keys' first dv
+// (with gate_wide gate[n * ld_gate + h * dv + d]), or null; r1, r2 [nh] or null; dist: 32-bit [nh, dist_len], the number
+// added to a score by head and distance (its last column for longer ones), or null; v_in_k: the values are the keys' first dv
 // elements; o_all: 32-bit [N, nh, nkv, dv] or null (then o is not written).
 MV_API int mv_attention_sink(const void* q, const void* pool, long long page_stride, const int* page_table,
                              int table_stride, int page_size, const int* positions, const int* seq_of,
                              const float* sinks, const float* gate, int ld_gate, void* o, int dtype, int N, int nh,
                              int nkv, int dk, int dv, float scale, float cap, int window, int keep_first,
-                             int head_tile, int chunk, const float* r1, const float* r2, int v_in_k, int gate_wide,
-                             float* o_all, cudaStream_t stream) {
+                             int head_tile, int chunk, const float* r1, const float* r2, const float* dist, int dist_len, int v_in_k,
+                             int gate_wide, float* o_all, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (dk < 1 || dk > AS_MAX_DIM || dv < 1 || dv > AS_MAX_DIM || nkv < 1 || nh % nkv || (page_size & (page_size - 1)) ||
-        (v_in_k && dv > dk) || (r1 && !r2))
+        (v_in_k && dv > dk) || (r1 && !r2) || (dist && dist_len < 1))
         return (int)cudaErrorInvalidValue;
     int page_shift = 0;
     while ((1 << page_shift) < page_size) ++page_shift;
@@ -402,12 +410,12 @@ MV_API int mv_attention_sink(const void* q, const void* pool, long long page_str
     if (pair)                                                                                                        \
         mv_launch(attention_sink_kernel<T, V, GTV, true>, blocks, AS_WARPS * 32, smem, stream, (const T*)q,          \
                   (const T*)pool, page_stride, page_table, table_stride, page_shift, positions, seq_of, sinks, gate, \
-                  ld_gate, (T*)o, N, nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2, v_in_k,         \
-                  gate_wide, o_all);                                                                                 \
+                  ld_gate, (T*)o, N, nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2, dist,           \
+                  dist_len, v_in_k, gate_wide, o_all);                                                               \
     else                                                                                                             \
     mv_launch(attention_sink_kernel<T, V, GTV, false>, blocks, AS_WARPS * 32, smem, stream, (const T*)q, (const T*)pool,    \
               page_stride, page_table, table_stride, page_shift, positions, seq_of, sinks, gate, ld_gate, (T*)o, N,  \
-              nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2, v_in_k, gate_wide, o_all);             \
+              nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2, dist, dist_len, v_in_k, gate_wide, o_all); \
     } while (0)
 #define AS_PICK(T, V)                                                                                                \
     do {                                                                                                             \

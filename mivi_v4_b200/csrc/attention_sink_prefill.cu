@@ -9,7 +9,9 @@
 // starts every row's maximum and denominator; the output is multiplied by the sigmoid of the row's gate;
 // with a chunked mask the walk starts at the first query's chunk and keys before a row's own chunk are masked.
 // Key and value sizes are run-time multiples of 16 up to the template's bounds.  Further parameters, as in
-// attention_sink.cu: a distance bias r1_h ln(1 + r2_h (i - j)) taken off the scores; values that are the keys' first dv
+// attention_sink.cu: a distance bias r1_h ln(1 + r2_h (i - j)) taken off the scores, or a table by head and
+// distance added to them (the head's row lies in shared memory where it is short; key blocks that lie wholly beyond it get
+// its last number); values that are the keys' first dv
 // elements; a gate per element instead of per head; every head's weights applied to every kv head's values (32-bit
 // results, for weights that are mixed between the heads afterwards).  SPLIT: a softmax weight enters the value
 // product as two bfloat16 numbers, the rounded weight and the rounding's remainder (two mma a tile), which
@@ -21,6 +23,7 @@ namespace {
 constexpr int QT = 64;          // queries per block
 constexpr int KB = 64;          // keys per block of the stream
 constexpr int NWARPS = 4;
+constexpr int DIST_SMEM = 2048; // numbers of a head's distance table that are kept in shared memory at most
 constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -60,7 +63,8 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
                               const float* __restrict__ sinks, const float* __restrict__ gate, int ld_gate,
                               __nv_bfloat16* __restrict__ o, int B, int nh, int nkv, int dk, int dv, float scale,
                               float cap, int window, int keep_first, int chunk, const float* __restrict__ r1,
-                              const float* __restrict__ r2, int v_in_k, int gate_wide, float* __restrict__ o_all) {
+                              const float* __restrict__ r2, const float* __restrict__ dist, int dist_len, int v_in_k,
+                              int gate_wide, float* __restrict__ o_all) {
     const int ldk = dk + 8, ldv = dv + 8;             // padded rows: conflict-free fragment loads
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(smem_raw);     // [2][KB][ldk]
@@ -77,6 +81,13 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
     const int h = o_all ? blockIdx.y / nkv : blockIdx.y, g = h / (nh / nkv);
     const int vg = o_all ? blockIdx.y - h * nkv : g;
     const float db1 = r1 ? r1[h] : 0.f, db2 = r1 ? r2[h] : 0.f;
+    const float* by_dist = dist ? dist + (size_t)h * dist_len : nullptr;
+    const float beyond = dist ? by_dist[dist_len - 1] : 0.f;
+    if (dist && dist_len <= DIST_SMEM) {
+        float* row = reinterpret_cast<float*>(vs + 2 * KB * ldv);       // (the loop's first barrier publishes it)
+        for (int i = threadIdx.x; i < dist_len; i += NWARPS * 32) row[i] = by_dist[i];
+        by_dist = row;
+    }
     const int row0 = cu[b] + tile * QT;
     const int rows_in_seq = cu[b + 1] - cu[b];
     const int nq = min(QT, rows_in_seq - tile * QT);
@@ -172,7 +183,10 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
         }
         // scale and cap, mask, then the running maximum of the two rows
         const int key0 = kb * KB;
-        const bool need_mask = r1 != nullptr || it < n_kept || key0 + KB - 1 > pos0 + warp * 16 ||
+        // the smallest distance between this warp's queries and the block's keys: from the table's last column on it is one number
+        const bool near = dist != nullptr && pos0 + warp * 16 - (key0 + KB - 1) < dist_len - 1;
+        const float add = dist != nullptr && !near ? beyond : 0.f;
+        const bool need_mask = r1 != nullptr || near || it < n_kept || key0 + KB - 1 > pos0 + warp * 16 ||
                                (chunk > 0 ? key0 < cs1 : (window > 0 && key0 <= pos0 + warp * 16 + 15 - window));
         float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
@@ -186,12 +200,14 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
                     const float x = sc * inv_cap, e2 = __expf(-2.0f * fabsf(x));
                     sc = copysignf(cap * __fdividef(1.0f - e2, 1.0f + e2), x);
                 }
+                sc += add;
                 if (need_mask) {
                     const int t = key0 + j * 8 + 2 * t4 + (e & 1);
                     const int p = (e < 2) ? p0 : p1;
                     if (t > p || (chunk > 0 ? t < ((e < 2) ? cs0 : cs1)
                                             : (window > 0 && t <= p - window && t >= keep_first))) sc = -INFINITY;
                     else if (r1) sc -= db1 * __logf(1.0f + db2 * (float)(p - t));
+                    else if (near) sc += by_dist[min(p - t, dist_len - 1)];
                 }
                 s[j][e] = sc;
             }
@@ -291,19 +307,21 @@ template <int DKM, int DVM, bool SPLIT>
 int launch(const void* q, const void* pool, long long page_stride, const int* page_table, int table_stride,
            int page_shift, const int* cu, const int* starts, const float* sinks, const float* gate, int ld_gate, void* o,
            int N, int B, int nh, int nkv, int dk, int dv, float scale, float cap, int window, int keep_first,
-           int chunk, const float* r1, const float* r2, int v_in_k, int gate_wide, float* o_all, cudaStream_t stream) {
-    const size_t smem = (size_t)2 * KB * (dk + 8 + dv + 8) * sizeof(__nv_bfloat16);
+           int chunk, const float* r1, const float* r2, const float* dist, int dist_len, int v_in_k, int gate_wide, float* o_all,
+           cudaStream_t stream) {
+    const size_t smem = (size_t)2 * KB * (dk + 8 + dv + 8) * sizeof(__nv_bfloat16) +
+                        (dist && dist_len <= DIST_SMEM ? dist_len * sizeof(float) : 0);
     static bool attr_set = false;
     if (!attr_set) {
         cudaFuncSetAttribute(attention_sink_prefill_kernel<DKM, DVM, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             (int)((size_t)2 * KB * (DKM + 8 + DVM + 8) * sizeof(__nv_bfloat16)));
+                             (int)((size_t)2 * KB * (DKM + 8 + DVM + 8) * sizeof(__nv_bfloat16) + DIST_SMEM * sizeof(float)));
         attr_set = true;
     }
     dim3 grid((N + QT - 1) / QT + B, o_all ? nh * nkv : nh);         // an upper bound of the tiles; spare blocks return at once
     attention_sink_prefill_kernel<DKM, DVM, SPLIT><<<grid, NWARPS * 32, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_stride, page_table, table_stride, page_shift, cu,
         starts, sinks, gate, ld_gate, (__nv_bfloat16*)o, B, nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2,
-        v_in_k, gate_wide, o_all);
+        dist, dist_len, v_in_k, gate_wide, o_all);
     return mv_launch_status();
 }
 
@@ -317,11 +335,11 @@ MV_API int mv_attention_sink_prefill(const void* q, const void* pool, long long 
                                      int table_stride, int page_size, const int* cu, const int* starts,
                                      const float* sinks, const float* gate, int ld_gate, void* o, int N, int B, int nh,
                                      int nkv, int dk, int dv, float scale, float cap, int window, int keep_first,
-                                     int chunk, const float* r1, const float* r2, int v_in_k, int gate_wide, float* o_all,
-                                     int split, cudaStream_t stream) {
+                                     int chunk, const float* r1, const float* r2, const float* dist, int dist_len, int v_in_k,
+                                     int gate_wide, float* o_all, int split, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (nkv < 1 || nh % nkv || (page_size & (page_size - 1)) || dk % 16 || dv % 16 || dk < 16 || dv < 16 || dk > 128 ||
-        dv > 128 || (v_in_k && dv > dk) || (r1 && !r2))
+        dv > 128 || (v_in_k && dv > dk) || (r1 && !r2) || (dist && (dist_len < 1 || r1)))
         return (int)cudaErrorInvalidValue;
     int page_shift = 0;
     while ((1 << page_shift) < page_size) ++page_shift;
@@ -330,10 +348,10 @@ MV_API int mv_attention_sink_prefill(const void* q, const void* pool, long long 
         if (split)                                                                                                   \
             return launch<A, C, true>(q, pool, page_stride, page_table, table_stride, page_shift, cu, starts, sinks, gate, \
                                       ld_gate, o, N, B, nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2, \
-                                      v_in_k, gate_wide, o_all, stream);                                             \
+                                      dist, dist_len, v_in_k, gate_wide, o_all, stream);                             \
         return launch<A, C, false>(q, pool, page_stride, page_table, table_stride, page_shift, cu, starts, sinks, gate, \
                                    ld_gate, o, N, B, nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2,    \
-                                   v_in_k, gate_wide, o_all, stream);                                                \
+                                   dist, dist_len, v_in_k, gate_wide, o_all, stream);                                \
     } while (0)
     if (dk <= 64 && dv <= 64) AS_GO(64, 64);
     if (dk <= 64) AS_GO(64, 128);

@@ -64,13 +64,18 @@ __device__ __forceinline__ float mv_block_sum(float v, float* scratch) {
     return scratch[32];
 }
 
-// The gated activations of a feed-forward: silu(g) * u, and g' * sigmoid(alpha g') * (u' + 1) with
-// g' = min(g, limit), u' = u cut off at -limit and limit.
+// The gated activations of a feed-forward: silu(g) * u, g' * sigmoid(alpha g') * (u' + 1) with
+// g' = min(g, limit), u' = u cut off at -limit and limit, and gelu(g) * u with the tanh form of gelu:
+// 0.5 (1 + tanh(y)) = 1 / (1 + e^(-2y)), y = sqrt(2 / pi) (g + 0.044715 g^3).
 __device__ __forceinline__ float mv_glu_silu(float g, float u) { return g / (1.0f + expf(-g)) * u; }
 __device__ __forceinline__ float mv_glu_clamped(float g, float u, float limit, float alpha) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+__device__ __forceinline__ float mv_glu_gelu(float g, float u) {
+    const float y2 = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);       // 2 sqrt(2 / pi) (g + 0.044715 g^3)
+    return g / (1.0f + expf(-y2)) * u;
 }
 
 // Loads 8 consecutive elements (16-byte aligned for bf16, 32-byte span for

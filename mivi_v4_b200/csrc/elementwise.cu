@@ -243,11 +243,12 @@ MV_API int mv_rmsnorm(const float* x, const float* w, void* y, int y_dtype, cons
 }
 
 // ------------------------------------------------------------------- swiglu
-// h[n, f] = silu(gate) * up, silu(a) = a / (1 + e^-a).  group == 0: gate = gu[n, f],
+// h[n, f] = silu(gate) * up, silu(a) = a / (1 + e^-a); with act 1 gelu(gate) * up, the tanh form of gelu.  group == 0: gate = gu[n, f],
 // up = gu[n, F + f] (the two halves end to end).  group == 16: the columns come in
 // groups of 16 gate values followed by the 16 up values of the same features.
 template <typename TO>
-__global__ void swiglu_kernel(const float* __restrict__ gu, TO* __restrict__ h, long long total, int F, int group) {
+__global__ void swiglu_kernel(const float* __restrict__ gu, TO* __restrict__ h, long long total, int F, int group,
+                              int act) {
     mv_pdl_begin();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
@@ -257,18 +258,18 @@ __global__ void swiglu_kernel(const float* __restrict__ gu, TO* __restrict__ h, 
     const int gb = group ? ga + group : F + f;
     const float a = gu[n * 2 * F + ga];
     const float b = gu[n * 2 * F + gb];
-    h[i] = mv_from_f32<TO>(a / (1.0f + expf(-a)) * b);
+    h[i] = mv_from_f32<TO>(act ? mv_glu_gelu(a, b) : mv_glu_silu(a, b));
 }
 
-MV_API int mv_swiglu(const float* gu, void* h, int h_dtype, int N, int F, int group, cudaStream_t stream) {
+MV_API int mv_swiglu(const float* gu, void* h, int h_dtype, int N, int F, int group, int act, cudaStream_t stream) {
     const long long total = (long long)N * F;
     if (total <= 0) return 0;
     const int threads = 256;
     const unsigned blocks = (unsigned)((total + threads - 1) / threads);
     if (h_dtype == MV_DT_BF16)
-        mv_launch(swiglu_kernel<__nv_bfloat16>, blocks, threads, 0, stream, gu, (__nv_bfloat16*)h, total, F, group);
+        mv_launch(swiglu_kernel<__nv_bfloat16>, blocks, threads, 0, stream, gu, (__nv_bfloat16*)h, total, F, group, act);
     else
-        mv_launch(swiglu_kernel<float>, blocks, threads, 0, stream, gu, (float*)h, total, F, group);
+        mv_launch(swiglu_kernel<float>, blocks, threads, 0, stream, gu, (float*)h, total, F, group, act);
     return mv_launch_status();
 }
 

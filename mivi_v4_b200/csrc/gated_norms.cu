@@ -1,5 +1,5 @@
 // Row-wise pieces that sit between matrix products: a layer norm (with or without a bias), a root-mean-square
-// norm over groups of a row followed by a gate, a root-mean-square norm whose result is added to
+// norm over groups of a row followed by a gate, a root-mean-square or layer norm whose result is added to
 // the residual stream, a clamped gated activation, a gate by a per-token table row, and the
 // rounding of 32-bit rows to the model's dtype.  Statistics and activations are 32-bit whatever
 // the output type.
@@ -158,41 +158,48 @@ MV_API int mv_rmsnorm_add(const float* y, const float* w, float* resid, int N, i
 
 // The same for a sublayer whose norm sits on its OUTPUT (x += norm(f(x))), where the output may be the
 // weighted sum of two branches, y = s1 y1 + s2 y2 (y2 null: y = s1 y1), and where the next sublayer reads
-// the completed row rounded to the model's dtype (rounded null: not written).
-template <typename TO>
-__global__ void rmsnorm_add_sum_kernel(const float* __restrict__ y1, float s1, const float* __restrict__ y2, float s2,
-                                       const float* __restrict__ w, float* __restrict__ resid, TO* __restrict__ rounded,
-                                       int H, float eps) {
+// the completed row rounded to the model's dtype (rounded null: not written).  CENTER: a layer norm, y less its mean
+// over the root of the mean squared deviation (+ eps), times w, plus b; else y over its root mean square, times w.
+template <typename TO, bool CENTER>
+__global__ void norm_add_sum_kernel(const float* __restrict__ y1, float s1, const float* __restrict__ y2, float s2,
+                                    const float* __restrict__ w, const float* __restrict__ b, float* __restrict__ resid,
+                                    TO* __restrict__ rounded, int H, float eps) {
     mv_pdl_begin();
     __shared__ float scratch[33];
     const size_t base = (size_t)blockIdx.x * H;
+    float mean = 0.f;
+    if (CENTER) {
+        float sum = 0.f;
+        for (int h = threadIdx.x; h < H; h += blockDim.x) sum += y2 ? fmaf(s2, y2[base + h], s1 * y1[base + h]) : s1 * y1[base + h];
+        mean = mv_block_sum(sum, scratch) / (float)H;
+    }
     float ss = 0.f;
     for (int h = threadIdx.x; h < H; h += blockDim.x) {
-        const float v = y2 ? fmaf(s2, y2[base + h], s1 * y1[base + h]) : s1 * y1[base + h];
+        const float v = (y2 ? fmaf(s2, y2[base + h], s1 * y1[base + h]) : s1 * y1[base + h]) - mean;
         ss = fmaf(v, v, ss);
     }
     const float scale = 1.0f / sqrtf(mv_block_sum(ss, scratch) / (float)H + eps);
     for (int h = threadIdx.x; h < H; h += blockDim.x) {
-        const float v = y2 ? fmaf(s2, y2[base + h], s1 * y1[base + h]) : s1 * y1[base + h];
-        const float r = resid[base + h] + v * scale * w[h];
+        const float v = (y2 ? fmaf(s2, y2[base + h], s1 * y1[base + h]) : s1 * y1[base + h]) - mean;
+        const float r = resid[base + h] + (CENTER ? fmaf(v * scale, w[h], b[h]) : v * scale * w[h]);
         resid[base + h] = r;
         if (rounded) rounded[base + h] = mv_from_f32<TO>(r);
     }
 }
 
-// The same with four values a load, a row's values kept in registers between the two passes: for rows of a
+// The same with four values a load, a row's values kept in registers between the passes: for rows of a
 // multiple of 4 and at most 8 values a thread, 16-byte aligned.
-template <typename TO>
+template <typename TO, bool CENTER>
 __global__ void __launch_bounds__(512)
-rmsnorm_add_sum_vec_kernel(const float* __restrict__ y1, float s1, const float* __restrict__ y2, float s2,
-                           const float* __restrict__ w, float* __restrict__ resid, TO* __restrict__ rounded, int H,
-                           float eps) {
+norm_add_sum_vec_kernel(const float* __restrict__ y1, float s1, const float* __restrict__ y2, float s2,
+                        const float* __restrict__ w, const float* __restrict__ b, float* __restrict__ resid,
+                        TO* __restrict__ rounded, int H, float eps) {
     mv_pdl_begin();
     __shared__ float scratch[33];
     const size_t base = (size_t)blockIdx.x * H;
     const int H4 = H >> 2;
     float4 v[2];
-    float ss = 0.f;
+    float sum = 0.f;
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         const int h4 = threadIdx.x + i * blockDim.x;
@@ -201,9 +208,18 @@ rmsnorm_add_sum_vec_kernel(const float* __restrict__ y1, float s1, const float* 
             const float4 a = reinterpret_cast<const float4*>(y1 + base)[h4];
             v[i] = make_float4(s1 * a.x, s1 * a.y, s1 * a.z, s1 * a.w);
             if (y2) {
-                const float4 b = reinterpret_cast<const float4*>(y2 + base)[h4];
-                v[i] = make_float4(fmaf(s2, b.x, v[i].x), fmaf(s2, b.y, v[i].y), fmaf(s2, b.z, v[i].z), fmaf(s2, b.w, v[i].w));
+                const float4 c = reinterpret_cast<const float4*>(y2 + base)[h4];
+                v[i] = make_float4(fmaf(s2, c.x, v[i].x), fmaf(s2, c.y, v[i].y), fmaf(s2, c.z, v[i].z), fmaf(s2, c.w, v[i].w));
             }
+            if (CENTER) sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+        }
+    }
+    const float mean = CENTER ? mv_block_sum(sum, scratch) / (float)H : 0.f;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        if (threadIdx.x + i * blockDim.x < H4) {
+            if (CENTER) v[i] = make_float4(v[i].x - mean, v[i].y - mean, v[i].z - mean, v[i].w - mean);
             ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss);
             ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
         }
@@ -215,32 +231,36 @@ rmsnorm_add_sum_vec_kernel(const float* __restrict__ y1, float s1, const float* 
         if (h4 < H4) {
             const float4 ww = reinterpret_cast<const float4*>(w)[h4];
             float4 r = reinterpret_cast<float4*>(resid + base)[h4];
-            r.x += v[i].x * scale * ww.x; r.y += v[i].y * scale * ww.y;
-            r.z += v[i].z * scale * ww.z; r.w += v[i].w * scale * ww.w;
+            if (CENTER) {
+                const float4 bb = reinterpret_cast<const float4*>(b)[h4];
+                r.x += fmaf(v[i].x * scale, ww.x, bb.x); r.y += fmaf(v[i].y * scale, ww.y, bb.y);
+                r.z += fmaf(v[i].z * scale, ww.z, bb.z); r.w += fmaf(v[i].w * scale, ww.w, bb.w);
+            } else {
+                r.x += v[i].x * scale * ww.x; r.y += v[i].y * scale * ww.y;
+                r.z += v[i].z * scale * ww.z; r.w += v[i].w * scale * ww.w;
+            }
             reinterpret_cast<float4*>(resid + base)[h4] = r;
             if (rounded) mv_store4(rounded + base + 4 * (size_t)h4, r.x, r.y, r.z, r.w);
         }
     }
 }
 
-MV_API int mv_rmsnorm_add_sum(const float* y1, float s1, const float* y2, float s2, const float* w, float* resid,
-                              void* rounded, int rounded_dtype, int N, int H, float eps, cudaStream_t stream) {
+// b (or null): the bias [H] of a layer norm; null: the root-mean-square norm
+MV_API int mv_norm_add_sum(const float* y1, float s1, const float* y2, float s2, const float* w, const float* b, float* resid,
+                           void* rounded, int rounded_dtype, int N, int H, float eps, cudaStream_t stream) {
     if (N <= 0) return 0;
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
-    const bool aligned = (((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)w | (uintptr_t)resid | (uintptr_t)rounded) & 15) == 0;
-    if (H % 4 == 0 && H / 4 <= 2 * threads && aligned) {
-        if (rounded && rounded_dtype == MV_DT_BF16)
-            mv_launch(rmsnorm_add_sum_vec_kernel<__nv_bfloat16>, N, threads, 0, stream, y1, s1, y2, s2, w, resid,
-                      (__nv_bfloat16*)rounded, H, eps);
-        else
-            mv_launch(rmsnorm_add_sum_vec_kernel<float>, N, threads, 0, stream, y1, s1, y2, s2, w, resid, (float*)rounded, H, eps);
-        return mv_launch_status();
-    }
-    if (rounded && rounded_dtype == MV_DT_BF16)
-        mv_launch(rmsnorm_add_sum_kernel<__nv_bfloat16>, N, threads, 0, stream, y1, s1, y2, s2, w, resid,
-                  (__nv_bfloat16*)rounded, H, eps);
-    else
-        mv_launch(rmsnorm_add_sum_kernel<float>, N, threads, 0, stream, y1, s1, y2, s2, w, resid, (float*)rounded, H, eps);
+    const bool aligned = (((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)w | (uintptr_t)b | (uintptr_t)resid | (uintptr_t)rounded) & 15) == 0;
+    const bool vec = H % 4 == 0 && H / 4 <= 2 * threads && aligned;
+#define NA_GO(K, TO, C) mv_launch(K<TO, C>, N, threads, 0, stream, y1, s1, y2, s2, w, b, resid, (TO*)rounded, H, eps)
+#define NA_PICK(TO)                                                                                                  \
+    do {                                                                                                             \
+        if (vec) { if (b) NA_GO(norm_add_sum_vec_kernel, TO, true); else NA_GO(norm_add_sum_vec_kernel, TO, false); } \
+        else { if (b) NA_GO(norm_add_sum_kernel, TO, true); else NA_GO(norm_add_sum_kernel, TO, false); }            \
+    } while (0)
+    if (rounded && rounded_dtype == MV_DT_BF16) NA_PICK(__nv_bfloat16); else NA_PICK(float);
+#undef NA_PICK
+#undef NA_GO
     return mv_launch_status();
 }
 

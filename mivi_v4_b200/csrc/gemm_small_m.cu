@@ -116,7 +116,7 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1
 // size), gridDim.y = row tiles.
 // TAIL 1 (RT == 3): the three row tiles of a warp are N rows apart, N counts channels, see ConvTail.
 // TAIL 2 (RT == 4): a tile is one head, see HeadTail.
-// TAIL 3 (RT == 2): mode 4, the clamped gated activation.
+// TAIL 3 (RT == 2): mode 4, the clamped gated activation.  TAIL 4 (RT == 2): mode 5, gelu(gate) * up.
 template <int NT, int RT, int UNROLL, int WARPS, int TAIL>
 __global__ void __launch_bounds__(WARPS * 32)
 gemm_small_m_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __restrict__ X,
@@ -432,12 +432,12 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __
             v *= 1.0f / sqrtf(ss * link.inv_dim + link.eps);
         }
         if (TAIL != 3 && bias && r < ROWS && n < N) v += bias[n];
-        if (TAIL == 3 || mode == 3) {
+        if (TAIL >= 3 || mode == 3) {
             // ROWS == 32: lanes 0-15 hold gate rows, lanes 16-31 the up rows of the same features
             const float up = __shfl_down_sync(0xffffffffu, v, 16);
             if (lane < 16 && n + 16 < N)
                 ((__nv_bfloat16*)out)[(size_t)m * ldo + (n >> 5) * 16 + lane] =
-                    __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v, up, bias[n], bias[N]) : mv_glu_silu(v, up));
+                    __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v, up, bias[n], bias[N]) : TAIL == 4 ? mv_glu_gelu(v, up) : mv_glu_silu(v, up));
         } else {
             float sq = 0.f;
             if (r < ROWS && n < N) {
@@ -518,7 +518,7 @@ MV_API int mv_gemm_small_m_tile_rows(int N, int mode) { return (N >= 32 * 2 * 14
 
 // mode: 0 store float32, 1 store bfloat16, 2 add into float32, 3 SwiGLU (W rows in
 // groups of 16 gate + 16 up; out is bfloat16 [M, N/2] with row stride ldo), 4 the clamped gated activation over
-// such rows (bias [N + 1]: a limit a row of W, then alpha).  Needs
+// such rows (bias [N + 1]: a limit a row of W, then alpha), 5 gelu (its tanh form) of the gate times up over such rows.  Needs
 // 1 <= M <= 64, K a multiple of 8, and 16-byte aligned operands.
 // scale_part (or null): [M][scale_stride] of which n_scale_part sums of squares per token; every token's
 // results are multiplied by rsqrt(sum / dim + eps) before bias and activation.  emit_x (or null, mode 2
@@ -531,7 +531,7 @@ MV_API int mv_gemm_small_m(const void* X, const void* W, const float* bias, void
                            int emit_stride, const void* next_w, long long next_bytes, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 64 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode >= 3 && (N % 32 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
+    if (mode < 0 || mode > 5 || (mode >= 3 && (N % 32 || (mode == 4 && !bias)))) return (int)cudaErrorInvalidValue;
     if (emit_x && (mode != 2 || ldo != N || !emit_g || !emit_part ||
                    emit_stride < (N + mv_gemm_small_m_tile_rows(N, 2) - 1) / mv_gemm_small_m_tile_rows(N, 2)))
         return (int)cudaErrorInvalidValue;
@@ -554,10 +554,14 @@ MV_API int mv_gemm_small_m(const void* X, const void* W, const float* bias, void
     const bool wide = mv_gemm_small_m_tile_rows(N, mode) == 32;
 #define MV_GO(NT, RT, U, WARPS)                                                                                                 \
     do {                                                                                                                        \
-        if constexpr (RT == 2)                                                                                                  \
+        if constexpr (RT == 2) {                                                                                                \
+            if (mode == 5)                                                                                                      \
+                return launch<NT, RT, U, WARPS, 4>(W, X, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{},            \
+                                                   Ahead{next_w, next_bytes}, stream);                                          \
             if (mode == 4)                                                                                                      \
                 return launch<NT, RT, U, WARPS, 3>(W, X, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{},            \
                                                    Ahead{next_w, next_bytes}, stream);                                          \
+        }                                                                                                                       \
         return launch<NT, RT, U, WARPS>(W, X, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, Ahead{next_w, next_bytes}, \
                                         stream);                                                                                \
     } while (0)

@@ -64,11 +64,11 @@ struct SmemLayout {
     static constexpr int TOTAL = TILE_BYTES + BAR_BYTES + 1024;      // 1024 for the manual alignment
 };
 
-template <int BN, int STAGES, bool CLAMP>
+template <int BN, int STAGES, int ACT>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                const float* __restrict__ bias, void* __restrict__ out, int mode, int M, int N, int K, int ldo,
-               const RowScale rs, int* __restrict__ err, const int* __restrict__ tile_group, int b_row_step,
+               const RowScale rs, const RowWeights rw, int* __restrict__ err, const int* __restrict__ tile_group, int b_row_step,
                int b_k_step) {
     using L = SmemLayout<BN, STAGES>;
     // A grouped product (tile_group not null): the rows of X are sorted by group and padded so that no tile of 128
@@ -158,7 +158,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 tmem_ld32(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)c0, r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 if (rs.part) scale_chunk(r, sc);
-                if (row < M) store_chunk<CLAMP>(r, row, n0 + c0, N, mode, bias, out, ldo);
+                if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, rw);
             }
         }
     }
@@ -190,11 +190,11 @@ struct WideLayout {
     static constexpr int TOTAL = TILE_BYTES + BAR_BYTES + 1024;
 };
 
-template <int STAGES, bool CLAMP>
+template <int STAGES, int ACT>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     const float* __restrict__ bias, void* __restrict__ out, int mode, int M, int N, int K, int ldo,
-                    const RowScale rs, int* __restrict__ err) {
+                    const RowScale rs, const RowWeights rw, int* __restrict__ err) {
     using L = WideLayout<STAGES>;
     constexpr int BN = L::BN;
     extern __shared__ unsigned char smem_raw[];
@@ -299,7 +299,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 tmem_ld32(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)(acc * BN + c0), r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 if (rs.part) scale_chunk(r, sc);
-                if (row < M) store_chunk<CLAMP>(r, row, n0 + c0, N, mode, bias, out, ldo);
+                if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, rw);
             }
             // this warp has read its lanes of the accumulator: hand it back
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -324,41 +324,41 @@ int sm_count() {
     return n;
 }
 
-template <int STAGES, bool CLAMP>
+template <int STAGES, int ACT>
 int launch_wide(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
-                const RowScale& rs, int* err, cudaStream_t stream) {
+                const RowScale& rs, const RowWeights& rw, int* err, cudaStream_t stream) {
     using L = WideLayout<STAGES>;
     CUtensorMap ma, mb;
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, N, K, L::BN, &mb)) return (int)cudaErrorInvalidValue;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(gemm_tc_wide_kernel<STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_wide_kernel<STAGES, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         attr_set = true;
     }
     const int tiles = ((M + BM - 1) / BM) * ((N + L::BN - 1) / L::BN);
     const int blocks = tiles < sm_count() ? tiles : sm_count();
-    gemm_tc_wide_kernel<STAGES, CLAMP><<<blocks, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, err);
+    gemm_tc_wide_kernel<STAGES, ACT><<<blocks, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, rw, err);
     return mv_launch_status();
 }
 
-template <int BN, int STAGES, bool CLAMP>
+template <int BN, int STAGES, int ACT>
 int launch(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
-           const RowScale& rs, int* err, cudaStream_t stream) {
+           const RowScale& rs, const RowWeights& rw, int* err, cudaStream_t stream) {
     using L = SmemLayout<BN, STAGES>;
     CUtensorMap ma, mb;
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, N, K, BN, &mb)) return (int)cudaErrorInvalidValue;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         attr_set = true;
     }
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
-    gemm_tc_kernel<BN, STAGES, CLAMP><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, err, nullptr, 0, 0);
+    gemm_tc_kernel<BN, STAGES, ACT><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, rs, rw, err, nullptr, 0, 0);
     return mv_launch_status();
 }
 
 // The grouped form: X [M, K] sorted by group, W [w_rows, w_cols] holding every group's matrix.
-template <int BN, int STAGES, bool CLAMP>
+template <int BN, int STAGES, int ACT>
 int launch_grouped(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo, int w_rows, int w_cols,
                    const int* tile_group, int b_row_step, int b_k_step, int* err, cudaStream_t stream) {
     using L = SmemLayout<BN, STAGES>;
@@ -366,11 +366,11 @@ int launch_grouped(const void* X, const void* W, const float* bias, void* out, i
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, w_rows, w_cols, BN, &mb)) return (int)cudaErrorInvalidValue;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         attr_set = true;
     }
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
-    gemm_tc_kernel<BN, STAGES, CLAMP><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, RowScale{}, err,
+    gemm_tc_kernel<BN, STAGES, ACT><<<grid, THREADS, L::TOTAL, stream>>>(ma, mb, bias, out, mode, M, N, K, ldo, RowScale{}, RowWeights{}, err,
                                                                    tile_group, b_row_step, b_k_step);
     return mv_launch_status();
 }
@@ -379,33 +379,41 @@ int launch_grouped(const void* X, const void* W, const float* bias, void* out, i
 
 // mode: 0 store float32, 1 store bfloat16, 2 add into float32, 3 SwiGLU (W rows in groups
 // of 16 gate + 16 up; out is bfloat16 [M, N/2] with row stride ldo), 4 the clamped gated activation over such rows
-// (bias [N + 1]: a limit a row of W, then alpha).  ``err`` points to a
+// (bias [N + 1]: a limit a row of W, then alpha), 5 gelu(gate) * up over such rows, 6 SwiGLU over such rows of experts
+// laid end to end, gate and up times row_w[row * ld_w + expert] first (RowWeights; no bias).  ``err`` points to a
 // device int that a block sets (1 producer, 2 MMA, 3 epilogue) if a wait ran out.
 // Needs K a multiple of 8 and 16-byte aligned operands.  scale_part (or null): the consuming end of a
 // carried norm, [M][scale_stride] with n_scale_part sums of squares a row over ``dim`` elements.
 MV_API int mv_gemm_tc(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N,
                       int K, int ldo, const float* scale_part, int n_scale_part, int scale_stride, int dim, float eps,
-                      int* err, cudaStream_t stream) {
+                      const float* row_w, int ld_w, int w_chunks, int w_experts, int* err, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
+    if (mode < 0 || mode > 6 || (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias)))) return (int)cudaErrorInvalidValue;
+    if (mode == 6 && (!row_w || bias || w_chunks < 1 || w_experts < 1)) return (int)cudaErrorInvalidValue;
+    const RowWeights rw = {row_w, ld_w, w_chunks, w_experts};
     if (scale_part && (n_scale_part <= 0 || n_scale_part > scale_stride || dim <= 0)) return (int)cudaErrorInvalidValue;
     RowScale rs = {};
     if (scale_part) rs = RowScale{scale_part, n_scale_part, scale_stride, 1.0f / (float)dim, eps};
-#define TC_GO(FN, ...) return mode == 4 ? FN<__VA_ARGS__, true>(X, W, bias, out, mode, M, N, K, ldo, rs, err, stream) \
-                                        : FN<__VA_ARGS__, false>(X, W, bias, out, mode, M, N, K, ldo, rs, err, stream)
+#define TC_ACT(FN, A, ...) FN<__VA_ARGS__, A>(X, W, bias, out, mode, M, N, K, ldo, rs, rw, err, stream)
+#define TC_GO(FN, ...)                                                                                                \
+    return mode == 4   ? TC_ACT(FN, ACT_CLAMPED, __VA_ARGS__)                                                         \
+           : mode == 5 ? TC_ACT(FN, ACT_GELU, __VA_ARGS__)                                                            \
+           : mode == 6 ? TC_ACT(FN, ACT_WEIGHTED, __VA_ARGS__)                                                        \
+                       : TC_ACT(FN, ACT_PLAIN, __VA_ARGS__)
     if (N <= 64) TC_GO(launch, 64, 4);
     // wide enough for 128 x 256 tiles to give every SM work: the persistent kernel
     const long long wide_tiles = (long long)((M + BM - 1) / BM) * ((N + 255) / 256);
     if (N >= 256 && wide_tiles >= 96) TC_GO(launch_wide, 4);
     TC_GO(launch, 128, 3);
 #undef TC_GO
+#undef TC_ACT
 }
 
 // The grouped product: the rows of X [M, K] are sorted by group and padded so that every tile of 128 rows belongs
 // to one group (tile_group [M / 128], negative for spare tiles); W [w_rows, w_cols] holds the groups' matrices one
 // below the other (b_row_step rows a group, b_k_step 0) or side by side along K (b_k_step columns a group, a
-// multiple of 8; b_row_step 0); N and K are ONE group's sizes.  Modes as mv_gemm_tc (no carried norm; bias, or mode 4's limits, are
+// multiple of 8; b_row_step 0); N and K are ONE group's sizes.  Modes 0 to 4 of mv_gemm_tc (no carried norm; bias, or mode 4's limits, are
 // the same for every group).
 // A tile's rows beyond its group's real rows hold whatever X holds there and give rows of ``out`` that nobody reads.
 MV_API int mv_gemm_tc_grouped(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
@@ -414,11 +422,11 @@ MV_API int mv_gemm_tc_grouped(const void* X, const void* W, const float* bias, v
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || M % BM || b_k_step % 8 || !tile_group || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
         return (int)cudaErrorInvalidValue;
-    if (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
+    if (mode > 4 || (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias)))) return (int)cudaErrorInvalidValue;
 #define TC_GO(BN, S)                                                                                                       \
-    return mode == 4 ? launch_grouped<BN, S, true>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, \
+    return mode == 4 ? launch_grouped<BN, S, ACT_CLAMPED>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, \
                                                    b_k_step, err, stream)                                                  \
-                     : launch_grouped<BN, S, false>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, \
+                     : launch_grouped<BN, S, ACT_PLAIN>(X, W, bias, out, mode, M, N, K, ldo, w_rows, w_cols, tile_group, b_row_step, \
                                                     b_k_step, err, stream)
     if (N <= 64) TC_GO(64, 4);
     TC_GO(128, 3);

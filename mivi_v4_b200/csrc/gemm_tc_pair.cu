@@ -99,11 +99,11 @@ __device__ __forceinline__ void arrive_remote(unsigned cluster_addr) {
     asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(cluster_addr) : "memory");
 }
 
-template <int STAGES, bool CLAMP>
+template <int STAGES, int ACT>
 __global__ void __launch_bounds__(PAIR_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     const float* __restrict__ bias, void* __restrict__ out, int mode, int M, int N, int K, int ldo,
-                    const PairLink link, int* __restrict__ err) {
+                    const PairLink link, const RowWeights rw, int* __restrict__ err) {
     using L = PairLayout<STAGES>;
     constexpr int BN = PAIR_BN;
     extern __shared__ unsigned char smem_raw[];
@@ -305,7 +305,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                         for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
                     }
-                    if (row < M) store_chunk<CLAMP>(r, row, n0 + c0, N, mode, bias, out, ldo);
+                    if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, rw);
                 }
             }
             // this warp has read its lanes of the accumulator: tell the leader's MMA warp
@@ -322,15 +322,15 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     }
 }
 
-template <int STAGES, bool CLAMP>
+template <int STAGES, int ACT>
 int launch_pair(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N, int K, int ldo,
-                const PairLink& link, int* err, cudaStream_t stream) {
+                const PairLink& link, const RowWeights& rw, int* err, cudaStream_t stream) {
     using L = PairLayout<STAGES>;
     CUtensorMap ma, mb;
     if (!tensor_map(X, M, K, BM, &ma) || !tensor_map(W, N, K, PAIR_BN / 2, &mb)) return (int)cudaErrorInvalidValue;
     static int max_pairs = 0;
     if (max_pairs == 0) {
-        cudaFuncSetAttribute(gemm_tc_pair_kernel<STAGES, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaFuncSetAttribute(gemm_tc_pair_kernel<STAGES, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         int dev = 0, sms = 148;
         cudaGetDevice(&dev);
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
@@ -345,7 +345,7 @@ int launch_pair(const void* X, const void* W, const float* bias, void* out, int 
         probe.attrs = pa;
         probe.numAttrs = 1;
         int n = 0;
-        if (cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel<STAGES, CLAMP>, &probe) != cudaSuccess || n <= 0) n = sms / 2;
+        if (cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel<STAGES, ACT>, &probe) != cudaSuccess || n <= 0) n = sms / 2;
         max_pairs = n < sms / 2 ? n : sms / 2;
         cudaGetLastError();
     }
@@ -363,7 +363,7 @@ int launch_pair(const void* X, const void* W, const float* bias, void* out, int 
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = mv_pdl_enabled() ? 2 : 1;
-    cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<STAGES, CLAMP>, ma, mb, bias, out, mode, M, N, K, ldo, link, err);
+    cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<STAGES, ACT>, ma, mb, bias, out, mode, M, N, K, ldo, link, rw, err);
     return mv_launch_status();
 }
 
@@ -373,11 +373,13 @@ int launch_pair(const void* X, const void* W, const float* bias, void* out, int 
 // does not take (the caller then uses mv_gemm_tc).
 MV_API int mv_gemm_tc_pair(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N,
                            int K, int ldo, const float* scale_part, int n_scale_part, int scale_stride, int dim,
-                           float eps, const float* emit_g, void* emit_x, float* emit_part, int emit_stride, int* err,
-                           cudaStream_t stream) {
+                           float eps, const float* emit_g, void* emit_x, float* emit_part, int emit_stride,
+                           const float* row_w, int ld_w, int w_chunks, int w_experts, int* err, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
+    if (mode < 0 || mode > 6 || (mode >= 3 && (N % 32 || ldo % 2 || (mode == 4 && !bias)))) return (int)cudaErrorInvalidValue;
+    if (mode == 6 && (!row_w || bias || w_chunks < 1 || w_experts < 1)) return (int)cudaErrorInvalidValue;
+    const RowWeights rw = {row_w, ld_w, w_chunks, w_experts};
     if (M <= BM || N < PAIR_BN / 2) return (int)cudaErrorInvalidValue;
     // an emitting product writes rows of 32 columns in 16-byte pieces: N in steps of 32, aligned buffers
     if (emit_x && (mode != 2 || ldo != N || N % 32 || !emit_g || !emit_part || emit_stride < (N + PAIR_BN - 1) / PAIR_BN ||
@@ -400,6 +402,10 @@ MV_API int mv_gemm_tc_pair(const void* X, const void* W, const float* bias, void
     }
     link.by_rows = (mode == 0 || mode == 2) && N % 32 == 0 && ldo % 4 == 0 && !(((uintptr_t)out | (uintptr_t)bias) & 15);
     if (emit_x && !link.by_rows) return (int)cudaErrorInvalidValue;
-    if (mode == 4) return launch_pair<6, true>(X, W, bias, out, mode, M, N, K, ldo, link, err, stream);
-    return launch_pair<6, false>(X, W, bias, out, mode, M, N, K, ldo, link, err, stream);
+#define PAIR_GO(A) return launch_pair<6, A>(X, W, bias, out, mode, M, N, K, ldo, link, rw, err, stream)
+    if (mode == 4) PAIR_GO(ACT_CLAMPED);
+    if (mode == 5) PAIR_GO(ACT_GELU);
+    if (mode == 6) PAIR_GO(ACT_WEIGHTED);
+    PAIR_GO(ACT_PLAIN);
+#undef PAIR_GO
 }

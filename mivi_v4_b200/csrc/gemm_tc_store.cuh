@@ -1,30 +1,48 @@
 // The epilogue of the tcgen05 matrix products: one row's 32 consecutive columns of the accumulator,
 // from registers to Y, in the mode asked for (0 store float32, 1 store bfloat16, 2 add into float32,
 // 3 SwiGLU over columns that alternate in groups of 16 gate and 16 up values, 4 the clamped gated activation over
-// such columns, ``bias`` then holding a limit a column and, after them, alpha).  Included inside the
-// including file's own namespace.
+// such columns, ``bias`` then holding a limit a column and, after them, alpha, 5 gelu (its tanh form) of the gate times up,
+// 6 SwiGLU of gate and up times a weight a row and an expert, see RowWeights).  Included inside the including file's
+// own namespace.
+// Mode 6: the columns are experts' gates and ups end to end, 32 * chunks of an expert; a row's weight for its expert e, w[row *
+// ld + e], multiplies gate and up before the activation (the expert's input carries it).  Columns after the last expert's
+// take 1.
+struct RowWeights {
+    const float* w;
+    int ld, chunks, n_experts;
+};
 // One row's 32 consecutive columns of the accumulator, from registers to Y, in the mode asked for.
-// CLAMP: mode 4, an instance of its own (the branch would cost the other modes registers).
-template <bool CLAMP>
+// ACT: an instance of its own for each of the modes 4, 5 and 6 (the branches would cost the other modes registers).
+enum { ACT_PLAIN = 0, ACT_CLAMPED = 1, ACT_GELU = 2, ACT_WEIGHTED = 3 };
+template <int ACT>
 __device__ __forceinline__ void store_chunk(const unsigned (&r)[32], int row, int n_base, int N, int mode,
-                                            const float* __restrict__ bias, void* __restrict__ out, int ldo) {
+                                            const float* __restrict__ bias, void* __restrict__ out, int ldo,
+                                            const RowWeights& rw) {
 
-        if (CLAMP || mode == 3) {
+        constexpr bool CLAMP = ACT == ACT_CLAMPED;
+        if (ACT != ACT_PLAIN || mode == 3) {
             // columns n_base .. +15 are gate, +16 .. +31 the up values of the same features
             if (n_base + 32 <= N) {
                 __nv_bfloat16* dst = (__nv_bfloat16*)out + (size_t)row * ldo + (n_base >> 1);
                 unsigned packed[8];
                 const float limit = CLAMP ? bias[n_base] : 0.f, alpha = CLAMP ? bias[N] : 0.f;
+                float wt = 1.f;
+                if (ACT == ACT_WEIGHTED) {
+                    const int e = (n_base >> 5) / rw.chunks;
+                    if (e < rw.n_experts) wt = rw.w[(size_t)row * rw.ld + e];
+                }
 #pragma unroll
                 for (int j = 0; j < 16; j += 2) {
                     float a0 = __uint_as_float(r[j]), a1 = __uint_as_float(r[j + 1]);
                     float b0 = __uint_as_float(r[j + 16]), b1 = __uint_as_float(r[j + 17]);
-                    if (!CLAMP && bias) {
+                    if (ACT == ACT_WEIGHTED) { a0 *= wt; a1 *= wt; b0 *= wt; b1 *= wt; }
+                    if ((ACT == ACT_PLAIN || ACT == ACT_GELU) && bias) {
                         a0 += bias[n_base + j]; a1 += bias[n_base + j + 1];
                         b0 += bias[n_base + j + 16]; b1 += bias[n_base + j + 17];
                     }
                     const __nv_bfloat162 v =
                         CLAMP ? __floats2bfloat162_rn(mv_glu_clamped(a0, b0, limit, alpha), mv_glu_clamped(a1, b1, limit, alpha))
+                        : ACT == ACT_GELU ? __floats2bfloat162_rn(mv_glu_gelu(a0, b0), mv_glu_gelu(a1, b1))
                               : __floats2bfloat162_rn(mv_glu_silu(a0, b0), mv_glu_silu(a1, b1));
                     packed[j >> 1] = *reinterpret_cast<const unsigned*>(&v);
                 }

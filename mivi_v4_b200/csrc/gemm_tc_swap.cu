@@ -377,7 +377,7 @@ gemm_tc_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                     for (int e = 0; e < 4; ++e)
                         if (n + e < N) v[e] += bias[n + e];
                 }
-                if (TAIL == 3 || mode == 3) {                // (TAIL 3: mode 4, the clamped gated activation)
+                if (TAIL >= 3 || mode == 3) {                // (TAIL 3: mode 4, the clamped gated activation; TAIL 4: mode 5, gelu)
                     // rows in groups of 16 gate + 16 up: of every 8 lanes the first 4 hold gate rows,
                     // the next 4 the up rows of the same features
                     float up[4];
@@ -388,7 +388,7 @@ gemm_tc_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                         for (int e = 0; e < 4; ++e)
                             o[e] = __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v[e], up[e], bias[n], bias[N])
-                                                                 : mv_glu_silu(v[e], up[e]));
+                                                      : TAIL == 4 ? mv_glu_gelu(v[e], up[e]) : mv_glu_silu(v[e], up[e]));
                     }
                 } else {
                     const size_t o = (size_t)m * ldo + n;
@@ -485,7 +485,7 @@ int launch(const void* X, const void* W, const float* bias, void* out, int mode,
 
 }  // namespace
 
-// Same contract as mv_gemm_small_m (modes 0-4, K a multiple of 8, 16-byte aligned operands;
+// Same contract as mv_gemm_small_m (modes 0-5, K a multiple of 8, 16-byte aligned operands;
 // scale_part / emit_x as there, with one sum per tile of 128 rows) for any M >= 1, plus the error
 // flag of the bounded waits.
 MV_API int mv_gemm_tc_swap(const void* X, const void* W, const float* bias, void* out, int mode, int M, int N,
@@ -494,7 +494,7 @@ MV_API int mv_gemm_tc_swap(const void* X, const void* W, const float* bias, void
                            const void* next_w, long long next_bytes, int* err, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
-    if (mode >= 3 && (N % 32 || (mode == 4 && !bias))) return (int)cudaErrorInvalidValue;
+    if (mode < 0 || mode > 5 || (mode >= 3 && (N % 32 || (mode == 4 && !bias)))) return (int)cudaErrorInvalidValue;
     if (emit_x && (mode != 2 || ldo != N || !emit_g || !emit_part || emit_stride < (N + BM - 1) / BM))
         return (int)cudaErrorInvalidValue;
     if (scale_part && (n_scale_part <= 0 || n_scale_part > scale_stride || dim <= 0)) return (int)cudaErrorInvalidValue;
@@ -521,6 +521,8 @@ MV_API int mv_gemm_tc_swap(const void* X, const void* W, const float* bias, void
         // multiprocessor).  Tiles of 256 tokens (one block a multiprocessor) measured slower at every size:
         // each block reads its own copy of X from the L2 cache, and that traffic grows with the tile.
         const int slices = k_slices(N, K, 2, (M + 127) / 128);
+        if (mode == 5)
+            return launch<128, 3, 4>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices);
         if (mode == 4)
             return launch<128, 3, 3>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices);
         return launch<128, 3>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices);
@@ -528,7 +530,10 @@ MV_API int mv_gemm_tc_swap(const void* X, const void* W, const float* bias, void
     const int slices = k_slices(N, K);
     const bool deep = slices == 1;
 #define MV_SWAP(BN, S, TAIL) launch<BN, S, TAIL>(X, W, bias, out, mode, M, N, K, ldo, link, ConvTail{}, HeadTail{}, ahead, err, stream, slices)
-#define MV_GO(BN) return mode == 4 ? (deep ? MV_SWAP(BN, 8, 3) : MV_SWAP(BN, 4, 3)) : (deep ? MV_SWAP(BN, 8, 0) : MV_SWAP(BN, 4, 0))
+#define MV_GO(BN)                                                                                                     \
+    return mode == 5   ? (deep ? MV_SWAP(BN, 8, 4) : MV_SWAP(BN, 4, 4))                                               \
+           : mode == 4 ? (deep ? MV_SWAP(BN, 8, 3) : MV_SWAP(BN, 4, 3))                                               \
+                       : (deep ? MV_SWAP(BN, 8, 0) : MV_SWAP(BN, 4, 0))
     if (M <= 16) MV_GO(16);
     if (M <= 32) MV_GO(32);
     MV_GO(64);

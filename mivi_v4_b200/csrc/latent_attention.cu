@@ -7,7 +7,8 @@
 // keys, and the values are the keys' first `rank` elements.  Nothing but c and r is cached or rebuilt.
 //
 //   * latent_prepare: from a token's projections, the root-mean-square norm of c (with a weight), the rotation of
-//     r and of the queries' rotated parts (element i of the rotated part pairs with i + rot/2), the row into its page;
+//     r and of the queries' rotated parts (element i of the rotated part pairs with i + rot/2; cos and sin may carry a factor),
+//     the row into its page;
 //     where the queries come through a latent of their own, that latent's norm instead of their rotation;
 //   * head_product: y[n, h, :] = W_h x[n, h, :] (or W_h^T), one small matrix per head: q -> qa (there with the rotation
 //     of the queries' last elements, if latent_prepare has not done it) and the output's way back (there with
@@ -32,7 +33,7 @@ latent_prepare_kernel(const float* __restrict__ proj, int ld, int q0, int c0, co
                       const float* __restrict__ inv_freq, const int* __restrict__ positions,
                       const int* __restrict__ seq_of, const int* __restrict__ page_table, int table_stride,
                       int page_shift, T* __restrict__ pool, long long page_stride, float* __restrict__ qa, int nh, int dim,
-                      int rot, int rank, int rot_dims, int cq0, int q_rank, const float* __restrict__ wq,
+                      int rot, int rank, int rot_dims, float amplitude, int cq0, int q_rank, const float* __restrict__ wq,
                       T* __restrict__ cq) {
     mv_pdl_begin();
     __shared__ float scratch[33];
@@ -44,8 +45,8 @@ latent_prepare_kernel(const float* __restrict__ proj, int ld, int q0, int c0, co
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float sn, cs;
         sincosf((float)pos * inv_freq[i], &sn, &cs);
-        rot_sn[i] = sn;
-        rot_cs[i] = cs;
+        rot_sn[i] = sn * amplitude;
+        rot_cs[i] = cs * amplitude;
     }
     const float* c = row + c0;
     float ss = 0.f;
@@ -92,8 +93,8 @@ MV_GUARD_SETTER(latent_attention)
 MV_API int mv_latent_prepare(const float* proj, int ld, int q0, int c0, const float* wc, float eps, const float* inv_freq,
                              const int* positions, const int* seq_of, const int* page_table, int table_stride,
                              int page_size, void* pool, long long page_stride, int dtype, float* qa, int N, int nh,
-                             int dim, int rot, int rank, int rot_dims, int cq0, int q_rank, const float* wq, void* cq,
-                             cudaStream_t stream) {
+                             int dim, int rot, int rank, int rot_dims, float amplitude, int cq0, int q_rank, const float* wq,
+                             void* cq, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (rot < 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > rot || rot > LA_MAX_ROT || rank < 1 || page_size < 1 || (page_size & (page_size - 1)))
         return (int)cudaErrorInvalidValue;
@@ -102,11 +103,11 @@ MV_API int mv_latent_prepare(const float* proj, int ld, int q0, int c0, const fl
     while ((1 << shift) < page_size) ++shift;
     if (dtype == MV_DT_BF16)
         mv_launch(latent_prepare_kernel<__nv_bfloat16>, N, 256, 0, stream, proj, ld, q0, c0, wc, eps, inv_freq, positions,
-                  seq_of, page_table, table_stride, shift, (__nv_bfloat16*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims, cq0,
-                  q_rank, wq, (__nv_bfloat16*)cq);
+                  seq_of, page_table, table_stride, shift, (__nv_bfloat16*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims,
+                  amplitude, cq0, q_rank, wq, (__nv_bfloat16*)cq);
     else
         mv_launch(latent_prepare_kernel<float>, N, 256, 0, stream, proj, ld, q0, c0, wc, eps, inv_freq, positions, seq_of,
-                  page_table, table_stride, shift, (float*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims, cq0, q_rank, wq,
+                  page_table, table_stride, shift, (float*)pool, page_stride, qa, nh, dim, rot, rank, rot_dims, amplitude, cq0, q_rank, wq,
                   (float*)cq);
     return mv_launch_status();
 }
@@ -128,6 +129,7 @@ struct RotTail {
     const float* inv_freq;
     const int* positions;
     int rot, rot_dims;
+    float amplitude;                // a factor on cos and sin
 };
 
 // the tail of tokens n0 .. n1 - 1 of head h: 32-bit in, 32-bit out (a tail is only asked for with 32-bit y)
@@ -142,6 +144,8 @@ __device__ __forceinline__ void rotate_tail(const RotTail& tail, const float* x,
         if (c < tail.rot_dims) {
             float sn, cs;
             sincosf((float)tail.positions[n] * tail.inv_freq[c < half ? c : c - half], &sn, &cs);
+            sn *= tail.amplitude;
+            cs *= tail.amplitude;
             v = c < half ? v * cs - src[c + half] * sn : v * cs + src[c - half] * sn;
         }
         y[(size_t)n * ldy + (size_t)h * hy + O + c] = mv_from_f32<TY>(v);
@@ -346,13 +350,13 @@ head_product_few_kernel(const float* __restrict__ x, long long ldx, int hx, cons
 // gate: with gate_heads one logit a head.  rot > 0 (32-bit y, y's rows at least O + rot wide): the tail, see above.
 MV_API int mv_head_product(const float* x, long long ldx, int hx, const void* w, int w_dtype, int transposed,
                            const float* gate, long long ldg, int gate_heads, void* y, int y_dtype, long long ldy, int hy,
-                           int N, int nh, int I, int O, int rot, int rot_dims, const float* inv_freq, const int* positions,
-                           cudaStream_t stream) {
+                           int N, int nh, int I, int O, int rot, int rot_dims, float amplitude, const float* inv_freq,
+                           const int* positions, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (nh < 1 || I < 1 || O < 1 || rot < 0 || rot_dims < 0 || rot_dims > rot || rot_dims % 2 ||
         (rot > 0 && (y_dtype != MV_DT_F32 || !positions || (rot_dims > 0 && !inv_freq))))
         return (int)cudaErrorInvalidValue;
-    const RotTail tail = {inv_freq, positions, rot, rot_dims};
+    const RotTail tail = {inv_freq, positions, rot, rot_dims, amplitude};
     const int more = rot > 0 ? 1 : 0;
     const size_t xs = sizeof(float) * (size_t)I * HF_T;
     const size_t elt = w_dtype == MV_DT_BF16 ? 2 : 4;

@@ -55,13 +55,18 @@ __device__ __forceinline__ int first_seen(int start, int window) { return window
 __global__ void __launch_bounds__(256)
 latent_query_kernel(const float* __restrict__ proj, int ld, int q0, const float* __restrict__ inv_freq,
                     const int* __restrict__ positions, __nv_bfloat16* __restrict__ q, int nh, int dim, int rot,
-                    int rot_dims) {
+                    int rot_dims, float amplitude) {
     mv_pdl_begin();
     const int n = blockIdx.x;
     const int dk = dim + rot, half = rot_dims >> 1;
     const float* row = proj + (size_t)n * ld + q0;
     __shared__ float sn_s[LQ_MAX_ROT / 2], cs_s[LQ_MAX_ROT / 2];          // a token's angles, once for all heads
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)positions[n] * inv_freq[i], &sn_s[i], &cs_s[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, cs;
+        sincosf((float)positions[n] * inv_freq[i], &sn, &cs);
+        sn_s[i] = sn * amplitude;
+        cs_s[i] = cs * amplitude;
+    }
     __syncthreads();
     __nv_bfloat16* dst = q + (size_t)n * nh * dk;
     for (int e = threadIdx.x; e < nh * dk; e += blockDim.x) {
@@ -334,13 +339,13 @@ int launch(const void* q, const void* kx, int ld_kx, int v0, const void* rk, con
 MV_GUARD_SETTER(latent_attention_prefill)
 
 // q [N, nh, dim + rot] bfloat16 from 32-bit rows `proj` (row stride ld, the queries from column q0), the first
-// rot_dims of every head's last rot elements turned by the angle positions[n] inv_freq[i] (i with i + rot_dims / 2).
+// rot_dims of every head's last rot elements turned by the angle positions[n] inv_freq[i] (i with i + rot_dims / 2), cos and sin times amplitude.
 MV_API int mv_latent_query(const float* proj, int ld, int q0, const float* inv_freq, const int* positions, void* q, int N,
-                           int nh, int dim, int rot, int rot_dims, cudaStream_t stream) {
+                           int nh, int dim, int rot, int rot_dims, float amplitude, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (rot_dims < 0 || rot_dims > rot || rot_dims > LQ_MAX_ROT || (rot_dims & 1) || (rot_dims && !inv_freq)) return (int)cudaErrorInvalidValue;
     mv_launch(latent_query_kernel, N, 256, 0, stream, proj, ld, q0, inv_freq, positions, (__nv_bfloat16*)q, nh, dim, rot,
-              rot_dims);
+              rot_dims, amplitude);
     return mv_launch_status();
 }
 

@@ -5,7 +5,7 @@
 // for the choice alone; some of the routed entries may be identity experts (no matrices: their output is their input).  The experts form `n_groups` equal groups of neighbours; a
 // group's score is the sum of its two largest s (of its only one, in groups of one); only experts of the
 // `keep` best groups can be chosen; the `top` largest s among those are chosen; their weights are s divided
-// by the sum of the chosen s (+ 1e-20).  Ties go to the lower index.  A shared expert's gate, sigmoid of one
+// by the sum of the chosen s (+ 1e-20), or s itself where they are not to be renormalized.  Ties go to the lower index.  A shared expert's gate, sigmoid of one
 // more logit, is written as one more column (a shared expert without a gate has none).  All of it is 32-bit.
 //
 // Output: a dense row of weights per token, [experts (+ 1)], zero for the experts that were not chosen, and
@@ -26,12 +26,12 @@ __device__ __forceinline__ void re_argmax(float& v, int& i) {
 // one warp a token.  z <- z + bias (or null).  mode 0: scores sigmoid(z); mode 1: scores softmax(z) over all E routed
 // entries; mode 2: scores z, the weights are softmax over the chosen z alone, times out_scale.  `correction`
 // (or null) is added to the scores for the CHOICE only; the weights are the chosen entries' own scores over their sum
-// (+ 1e-20), times out_scale.  The last n_identity of the E entries are identity experts: the dense row is laid out
+// (+ 1e-20) (without renorm: the scores themselves), times out_scale.  The last n_identity of the E entries are identity experts: the dense row is laid out
 // [E - n_identity experts | the shared gate, if any | n_identity identity weights].
 __global__ void __launch_bounds__(128)
 route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int* __restrict__ pick,
              float* __restrict__ pick_w, int N, int E, int n_groups, int keep, int top, int shared_gate, int mode,
-             const float* __restrict__ correction, float out_scale, int n_identity, const float* __restrict__ bias) {
+             const float* __restrict__ correction, float out_scale, int n_identity, const float* __restrict__ bias, int renorm) {
     mv_pdl_begin();
     extern __shared__ float re_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -112,7 +112,7 @@ route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int
         w = lane < top ? expf(w - best) : 0.f;
         sum = mv_warp_sum(w);
     }
-    w *= out_scale / (mode == 2 ? sum : sum + 1e-20f);
+    w *= mode == 2 ? out_scale / sum : (renorm ? out_scale / (sum + 1e-20f) : out_scale);
     if (lane < top) {
         pick_w[(size_t)n * top + lane] = w;
         const int i = pick[(size_t)n * top + lane];
@@ -123,7 +123,7 @@ route_kernel(const float* __restrict__ z, int ld, float* __restrict__ dense, int
 // z [N, >= E (+ 1)] with row stride ld; dense [N, E (+ 1)]; pick, pick_w [N, top]; correction, bias [E] or null.
 MV_API int mv_route(const float* z, int ld, float* dense, int* pick, float* pick_w, int N, int E, int n_groups,
                     int keep, int top, int shared_gate, int mode, const float* correction, float out_scale,
-                    int n_identity, const float* bias, cudaStream_t stream) {
+                    int n_identity, const float* bias, int renorm, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (E < 1 || E > RE_MAX_EXPERTS || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups || top < 1 ||
         top > 32 || top > keep * (E / n_groups) || n_identity < 0 || n_identity > E || mode < 0 || mode > 2)
@@ -131,7 +131,7 @@ MV_API int mv_route(const float* z, int ld, float* dense, int* pick, float* pick
     const int warps = 4;
     const size_t smem = sizeof(float) * warps * (size_t)(2 * E + n_groups);
     mv_launch(route_kernel, (N + warps - 1) / warps, warps * 32, smem, stream, z, ld, dense, pick, pick_w, N, E,
-              n_groups, keep, top, shared_gate, mode, correction, out_scale, n_identity, bias);
+              n_groups, keep, top, shared_gate, mode, correction, out_scale, n_identity, bias, renorm);
     return mv_launch_status();
 }
 
@@ -170,12 +170,13 @@ MV_API int mv_identity_experts(const void* h, int dtype, const float* dense, int
 // (expert e owns [e * ff, (e + 1) * ff), a shared expert the `shared_ff` columns after them, with the weight of
 // column E, or 1 where it has no gate).  gu [N, 2 * F] holds an expert's gates and ups together, [e * 2 ff, (e + 1) * 2 ff): alternating in
 // groups of 16 columns (16 gates, their 16 ups, ...) where `group` says so, else the gates, then the ups; the
-// shared expert's block follows with `shared_group`.  Where the weight is zero nothing is computed.
+// shared expert's block follows with `shared_group`.  Where the weight is zero nothing is computed.  on_input: the weight
+// multiplies the expert's INPUT, hid = act(w gate, w up) (gate and up are linear in it).
 template <typename TO>
 __global__ void __launch_bounds__(256)
 routed_glu_kernel(const float* __restrict__ gu, const float* __restrict__ dense, TO* __restrict__ hid, long long total,
-                  int F, int E, int ff, int shared_ff, int cols, int group, int shared_group, int shared_gate, float limit,
-                  float shared_limit, float alpha) {
+                  int F, int E, int ff, int shared_ff, int cols, int group, int shared_group, int shared_gate, int on_input,
+                  float limit, float shared_limit, float alpha) {
     mv_pdl_begin();
     const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
@@ -188,16 +189,18 @@ routed_glu_kernel(const float* __restrict__ gu, const float* __restrict__ dense,
         const int cc = c - e * ff, width = e < E ? ff : shared_ff, grp = e < E ? group : shared_group;
         const float* blk = gu + n * 2 * F + (size_t)e * 2 * ff;
         const int gi = grp ? (cc / grp) * 2 * grp + cc % grp : cc;
-        const float g = blk[gi], u = blk[gi + (grp ? grp : width)];
-        out = w * (limit > 0.f ? mv_glu_clamped(g, u, e < E ? limit : shared_limit, alpha) : mv_glu_silu(g, u));
+        const bool first = on_input && e < E;                // (a shared expert's gate is always on its output)
+        const float wi = first ? w : 1.f;
+        const float g = wi * blk[gi], u = wi * blk[gi + (grp ? grp : width)];
+        out = (first ? 1.f : w) * (limit > 0.f ? mv_glu_clamped(g, u, e < E ? limit : shared_limit, alpha) : mv_glu_silu(g, u));
     }
     hid[idx] = mv_from_f32<TO>(out);
 }
 
 // extra_cols: columns of a dense row after the experts' (and the shared gate's) that belong to others
 MV_API int mv_routed_glu(const float* gu, const float* dense, void* hid, int hid_dtype, int N, int E, int ff,
-                         int shared_ff, int group, int shared_group, int extra_cols, int shared_gate, float limit,
-                         float shared_limit, float alpha, cudaStream_t stream) {
+                         int shared_ff, int group, int shared_group, int extra_cols, int shared_gate, int on_input,
+                         float limit, float shared_limit, float alpha, cudaStream_t stream) {
     if (N <= 0) return 0;
     const int F = E * ff + shared_ff, cols = E + (shared_ff && shared_gate ? 1 : 0) + extra_cols;
     if ((group && ff % group) || (shared_group && shared_ff % shared_group)) return (int)cudaErrorInvalidValue;
@@ -205,10 +208,10 @@ MV_API int mv_routed_glu(const float* gu, const float* dense, void* hid, int hid
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (hid_dtype == MV_DT_BF16)
         mv_launch(routed_glu_kernel<__nv_bfloat16>, blocks, 256, 0, stream, gu, dense, (__nv_bfloat16*)hid, total, F, E,
-                  ff, shared_ff, cols, group, shared_group, shared_gate, limit, shared_limit, alpha);
+                  ff, shared_ff, cols, group, shared_group, shared_gate, on_input, limit, shared_limit, alpha);
     else
         mv_launch(routed_glu_kernel<float>, blocks, 256, 0, stream, gu, dense, (float*)hid, total, F, E, ff, shared_ff, cols,
-                  group, shared_group, shared_gate, limit, shared_limit, alpha);
+                  group, shared_group, shared_gate, on_input, limit, shared_limit, alpha);
     return mv_launch_status();
 }
 
@@ -241,12 +244,13 @@ expert_rank_kernel(const int* __restrict__ pick, int total, int* __restrict__ ra
     if (tid == 0) counts[e] = base;
 }
 
-// place[entry] = (entries of the experts before its own) + its rank; the token's row is copied there.
+// place[entry] = (entries of the experts before its own) + its rank; the token's row is copied there (in_w not null: times
+// the entry's weight).
 template <typename T>
 __global__ void __launch_bounds__(128)
 expert_gather_kernel(const int* __restrict__ pick, const int* __restrict__ rank, const int* __restrict__ counts,
-                     const int* __restrict__ offsets, const T* __restrict__ x, int top, int H, int* __restrict__ place,
-                     T* __restrict__ xs) {
+                     const int* __restrict__ offsets, const T* __restrict__ x, const float* __restrict__ in_w, int top, int H,
+                     int* __restrict__ place, T* __restrict__ xs) {
     mv_pdl_begin();
     __shared__ float scratch[33];
     const int idx = blockIdx.x;
@@ -262,9 +266,15 @@ expert_gather_kernel(const int* __restrict__ pick, const int* __restrict__ rank,
     if (threadIdx.x == 0) place[idx] = p;
     const T* src = x + (size_t)(idx / top) * H;
     T* dst = xs + (size_t)p * H;
+    if (in_w) {
+        const float w = in_w[idx];
+        for (int h = threadIdx.x; h < H; h += blockDim.x) dst[h] = mv_from_f32<T>(w * mv_to_f32(src[h]));
+        return;
+    }
     for (int h = threadIdx.x; h < H; h += blockDim.x) dst[h] = src[h];
 }
 
+// pick_w null: every chosen expert's result counts as it is.
 // out[n, :] (+)= sum_k w[n, k] ys[place[n * top + k], :] + gate[n] shared[n, :], the choices in their order
 __global__ void __launch_bounds__(256)
 expert_combine_kernel(const float* __restrict__ ys, const int* __restrict__ place, const float* __restrict__ pick_w,
@@ -275,7 +285,7 @@ expert_combine_kernel(const float* __restrict__ ys, const int* __restrict__ plac
     for (int h = threadIdx.x; h < H; h += blockDim.x) {
         float sum = 0.f;
         for (int k = 0; k < top; ++k)
-            sum = fmaf(pick_w[(size_t)n * top + k], ys[(size_t)place[(size_t)n * top + k] * H + h], sum);
+            sum = fmaf(pick_w ? pick_w[(size_t)n * top + k] : 1.f, ys[(size_t)place[(size_t)n * top + k] * H + h], sum);
         if (shared) sum = fmaf(gate ? gate[(size_t)n * ld_gate] : 1.f, shared[(size_t)n * H + h], sum);
         float* o = out + (size_t)n * H + h;
         *o = accumulate ? *o + sum : sum;
@@ -292,13 +302,13 @@ MV_API int mv_expert_rank(const int* pick, int total, int E, int* rank, int* cou
 // x [N, H] in `dtype` -> xs [N * top, H] sorted by expert; place [N * top] says where each entry went
 // offsets (or null): where every expert's run of rows starts (mv_expert_tiles), instead of the plain sums of counts
 MV_API int mv_expert_gather(const int* pick, const int* rank, const int* counts, const int* offsets, const void* x,
-                            int dtype, int N, int top, int H, int* place, void* xs, cudaStream_t stream) {
+                            int dtype, const float* in_w, int N, int top, int H, int* place, void* xs, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (dtype == MV_DT_BF16)
         mv_launch(expert_gather_kernel<__nv_bfloat16>, N * top, 128, 0, stream, pick, rank, counts, offsets,
-                  (const __nv_bfloat16*)x, top, H, place, (__nv_bfloat16*)xs);
+                  (const __nv_bfloat16*)x, in_w, top, H, place, (__nv_bfloat16*)xs);
     else
-        mv_launch(expert_gather_kernel<float>, N * top, 128, 0, stream, pick, rank, counts, offsets, (const float*)x, top, H,
+        mv_launch(expert_gather_kernel<float>, N * top, 128, 0, stream, pick, rank, counts, offsets, (const float*)x, in_w, top, H,
                   place, (float*)xs);
     return mv_launch_status();
 }

@@ -35,7 +35,7 @@ _SIGNATURES = {
         "mv_embed_link": [_P, _I, _P, _P, _I, _I, _P, _P, _P, _I, _P],
         "mv_embed_link_partials": [_I],
         "mv_rmsnorm": [_P, _P, _P, _I, _P, _I, _I, _F, _P],
-        "mv_swiglu": [_P, _P, _I, _I, _I, _I, _P],
+        "mv_swiglu": [_P, _P, _I, _I, _I, _I, _I, _P],
         "mv_copy_to_host": [_P, _P, _Q, _P],
         "mv_delay": [_Q, _P],
         "mv_gemm_simt": [_P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
@@ -59,16 +59,16 @@ _SIGNATURES = {
         "mv_decay_scan_chunked": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _F, _F, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I,
                                   _I, _I, _I, _P],
         "mv_qkv_prepare_wide": [_P, _I, _P, _P, _F, _I, _P, _P, _P, _P, _I, _I, _P, _Q, _P, _I, _I, _I, _I, _I, _I, _I,
-                                _F, _P],
+                                _F, _F, _F, _P],
         "mv_attention_sink": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _I,
-                              _I, _I, _P, _P, _I, _I, _P, _P],
+                              _I, _I, _P, _P, _P, _I, _I, _I, _P, _P],
         "mv_mix_heads": [_P, _P, _P, _I, _I, _I, _I, _I, _P],
         "mv_block_gates": [_P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P],
         "mv_gated_recurrence": [_P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P],
         "mv_scaled_add_norm": [_P, _F, _P, _F, _P, _P, _P, _F, _P, _I, _I, _I, _P],
         "mv_embed_scaled_pos": [_P, _I, _P, _F, _P, _P, _P, _P, _I, _I, _I, _P],
         "mv_softcap": [_P, _Q, _F, _P],
-        "mv_rmsnorm_add_sum": [_P, _F, _P, _F, _P, _P, _P, _I, _I, _I, _F, _P],
+        "mv_norm_add_sum": [_P, _F, _P, _F, _P, _P, _P, _P, _I, _I, _I, _F, _P],
         "mv_scalar_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I,
                            _P],
         "mv_scalar_chunks": [_I, _I],
@@ -78,20 +78,20 @@ _SIGNATURES = {
         "mv_causal_conv": [_P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
         "mv_ssm_decode_prepare": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
         "mv_step_size": [_P, _I, _P, _P, _P, _P, _I, _I, _P],
-        "mv_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _P, _P],
-        "mv_routed_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
+        "mv_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _P, _I, _P],
+        "mv_routed_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
         "mv_scale_expert_columns": [_P, _I, _P, _I, _I, _I, _I, _I, _I, _P],
         "mv_identity_experts": [_P, _I, _P, _I, _I, _I, _P, _I, _I, _I, _P],
         "mv_embed_bigram": [_P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _Q, _Q, _P],
         "mv_add_rows_vector": [_P, _P, _P, _I, _I, _P],
-        "mv_latent_prepare": [_P, _I, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _P, _Q, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I,
+        "mv_latent_prepare": [_P, _I, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _P, _Q, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I,
                               _P, _P, _P],
-        "mv_head_product": [_P, _Q, _I, _P, _I, _I, _P, _Q, _I, _P, _I, _Q, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P],
+        "mv_head_product": [_P, _Q, _I, _P, _I, _I, _P, _Q, _I, _P, _I, _Q, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P],
         "mv_latent_attention": [_P, _P, _Q, _I, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P],
         "mv_delta_scan_long": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _F, _F, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
         "mv_delta_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _F, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
         "mv_expert_rank": [_P, _I, _I, _P, _P, _P],
-        "mv_expert_gather": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P],
+        "mv_expert_gather": [_P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _P, _P, _P],
         "mv_expert_tiles": [_P, _I, _I, _P, _P, _I, _P],
         "mv_expert_combine": [_P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P],
         "mv_sample": [_P, _Q, _P, _I, _I, _F, _I, _F, _F, _F, _F, _F, _P, _P, _UQ, _P, _P, _P, _P, _P, _P, _P, _P],
@@ -102,9 +102,9 @@ _SIGNATURES = {
         "mv_gemm_small_m_shortconv": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _Q, _P],
         "mv_gemm_small_m_heads": [_P, _P, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _Q, _P, _I, _I, _I, _I,
                                   _P, _I, _I, _I, _F, _P, _Q, _P],
-        "mv_gemm_tc": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P],
+        "mv_gemm_tc": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P],
         "mv_gemm_tc_grouped": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P],
-        "mv_gemm_tc_pair": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P, _P, _I, _P, _P],
+        "mv_gemm_tc_pair": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P, _P, _I, _P, _I, _I, _I, _P, _P],
         "mv_gemm_tc_swap": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P, _P, _I, _P, _Q, _P, _P],
         "mv_gemm_tc_swap_shortconv": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _Q,
                                       _P, _P],
@@ -112,11 +112,11 @@ _SIGNATURES = {
                                   _P, _I, _I, _I, _F, _P, _Q, _P, _P],
         "mv_attention_prefill": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
         "mv_attention_sink_prefill": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I,
-                                      _I, _I, _P, _P, _I, _I, _P, _I, _P],
+                                      _I, _I, _P, _P, _P, _I, _I, _I, _P, _I, _P],
         "mv_attention_decode_tc": [_P, _P, _Q, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _P, _P],
         "mv_attention_prefill_tc": [_P, _P, _Q, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
         "mv_latent_attention_decode": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P, _P],
-        "mv_latent_query": [_P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+        "mv_latent_query": [_P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P],
         "mv_latent_gather": [_P, _Q, _P, _I, _I, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P],
         "mv_latent_attention_prefill": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P],
     },
@@ -540,16 +540,18 @@ def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
     return x
 
 
-def rmsnorm_add_sum(y1: torch.Tensor, w: torch.Tensor, eps: float, resid: torch.Tensor, *, s1: float = 1.0,
-                    y2: Optional[torch.Tensor] = None, s2: float = 1.0, rounded: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """resid += y / sqrt(mean(y^2) + eps) * w with y = s1 * y1 (+ s2 * y2), all float32; ``rounded`` also gets
+def norm_add_sum(y1: torch.Tensor, w: torch.Tensor, eps: float, resid: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
+                 s1: float = 1.0, y2: Optional[torch.Tensor] = None, s2: float = 1.0,
+                 rounded: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """resid += norm(y) with y = s1 * y1 (+ s2 * y2), all float32: the root-mean-square norm y / sqrt(mean(y^2) + eps) * w,
+    or with ``bias`` [H] the layer norm (y - mean) / sqrt(mean((y - mean)^2) + eps) * w + bias; ``rounded`` also gets
     the completed rows in its own dtype (what the next sublayer multiplies)."""
     N, H = y1.shape
-    _check(_fn("core", "mv_rmsnorm_add_sum")(
-        _need(y1, "rmsnorm_add_sum y1", torch.float32), float(s1), _need(y2, "rmsnorm_add_sum y2", torch.float32, (N, H), True),
-        float(s2), _need(w, "rmsnorm_add_sum weight", torch.float32, (H,)),
+    _check(_fn("core", "mv_norm_add_sum")(
+        _need(y1, "norm_add_sum y1", torch.float32), float(s1), _need(y2, "norm_add_sum y2", torch.float32, (N, H), True),
+        float(s2), _need(w, "norm_add_sum weight", torch.float32, (H,)), _need(bias, "norm_add_sum bias", torch.float32, (H,), True),
         _need(resid, "residual stream", torch.float32, (N, H)), _need(rounded, "rounded rows", None, (N, H), True),
-        _dt(rounded) if rounded is not None else F32, N, H, float(eps), _stream()), "mv_rmsnorm_add_sum")
+        _dt(rounded) if rounded is not None else F32, N, H, float(eps), _stream()), "mv_norm_add_sum")
     account(N * H * (12 + (4 if y2 is not None else 0) + (rounded.element_size() if rounded is not None else 0)))
     return resid
 
@@ -781,14 +783,14 @@ ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_CHOSEN_SOFTMAX = 0, 1, 2
 def route(z: torch.Tensor, dense: torch.Tensor, pick: torch.Tensor, pick_w: torch.Tensor, n_experts: int,
           n_groups: int, keep: int, top: int, shared_gate: bool, *, mode: int = ROUTE_SIGMOID,
           correction: Optional[torch.Tensor] = None, out_scale: float = 1.0, n_identity: int = 0,
-          bias: Optional[torch.Tensor] = None) -> None:
+          bias: Optional[torch.Tensor] = None, renormalize: bool = True) -> None:
     """Router of a mixture of experts from float32 logits ``z`` [N, routed (+ 1)] (``bias`` [routed] is added to them
     first): scores sigmoid(z), or with ``ROUTE_SOFTMAX`` softmax(z) over all routed entries, or with
     ``ROUTE_CHOSEN_SOFTMAX`` the logits themselves, the weights then being softmax over the chosen logits alone, times
     ``out_scale``; the entries
     form ``n_groups`` equal groups of neighbours whose score is the sum of their two largest scores; among the
     entries of the ``keep`` best groups the ``top`` largest are chosen, with weights score / (sum of the chosen
-    scores + 1e-20) * ``out_scale``.  ``correction`` [routed] is added to the scores for the choice only.
+    scores + 1e-20) * ``out_scale``, or without ``renormalize`` score * ``out_scale``.  ``correction`` [routed] is added to the scores for the choice only.
     ``n_experts`` counts all routed entries; its last ``n_identity`` are identity experts.  ``dense``
     [N, routed (+ 1)] gets a row of weights (zero where not chosen), laid out [experts | with ``shared_gate``
     sigmoid of the last logit | identity experts]; ``pick`` / ``pick_w`` [N, top] the lists (routed indices)."""
@@ -804,7 +806,8 @@ def route(z: torch.Tensor, dense: torch.Tensor, pick: torch.Tensor, pick_w: torc
         zp, ldz, _need(dense, "route weights", torch.float32, (N, cols)), _need(pick, "route picks", torch.int32, (N, top)),
         _need(pick_w, "route pick weights", torch.float32, (N, top)), N, E, int(n_groups), int(keep), int(top),
         int(bool(shared_gate)), int(mode), _need(correction, "route correction", torch.float32, (E,), True),
-        float(out_scale), int(n_identity), _need(bias, "router bias", torch.float32, (E,), True), _stream()), "mv_route")
+        float(out_scale), int(n_identity), _need(bias, "router bias", torch.float32, (E,), True), int(bool(renormalize)),
+        _stream()), "mv_route")
     account(N * cols * 8)
 
 
@@ -825,14 +828,15 @@ def identity_experts(h: torch.Tensor, dense: torch.Tensor, col0: int, n_cols: in
 
 def routed_glu(gu: torch.Tensor, dense: torch.Tensor, hid: torch.Tensor, n_experts: int, ff: int, shared_ff: int,
                group: int = 0, shared_group: int = 0, extra_cols: int = 0, shared_gate: bool = True, limit: float = 0.0,
-               shared_limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
+               shared_limit: float = 0.0, alpha: float = 0.0, on_input: bool = False) -> torch.Tensor:
     """hid[n, c] = weight(n, expert of column c) * silu(gate[n, c]) * up[n, c] over the columns of all experts end to
     end (then a shared expert's), from ``gu`` [N, 2 * F] float32 and the router's dense weights; nothing is computed
     where the weight is zero.  ``gu`` holds each expert's gates and ups together, [e * 2 ff, (e + 1) * 2 ff): the gates,
     then the ups, or with ``group`` 16 alternating in groups of 16 columns; the shared expert's block likewise with
     ``shared_group``.  Without ``shared_gate`` the dense weights have no column for the shared expert and its weight
     is 1.  ``limit`` > 0: the clamped gated activation of :func:`glu_clamped` instead of silu(gate) * up, with
-    ``shared_limit`` for the shared expert."""
+    ``shared_limit`` for the shared expert.  ``on_input``: the weight multiplies the expert's input, so gate and up
+    each carry it before the activation."""
     N, F = hid.shape
     if F != n_experts * ff + shared_ff:
         raise KernelError(f"routed_glu: {F} columns for {n_experts} experts of {ff} and a shared one of {shared_ff}")
@@ -842,7 +846,8 @@ def routed_glu(gu: torch.Tensor, dense: torch.Tensor, hid: torch.Tensor, n_exper
         _need(gu, "routed_glu input", torch.float32, (N, 2 * F)),
         _need(dense, "route weights", torch.float32, (N, n_experts + (1 if shared_ff and shared_gate else 0) + extra_cols)),
         _need(hid, "routed_glu out"), _dt(hid), N, int(n_experts), int(ff), int(shared_ff), int(group), int(shared_group),
-        int(extra_cols), int(bool(shared_gate)), float(limit), float(shared_limit), float(alpha), _stream()), "mv_routed_glu")
+        int(extra_cols), int(bool(shared_gate)), int(bool(on_input)), float(limit), float(shared_limit), float(alpha), _stream()),
+        "mv_routed_glu")
     account(N * F * (8 + hid.element_size()))
     return hid
 
@@ -874,13 +879,14 @@ def grouped_tiles(n_entries: int, n_experts: int) -> int:
 
 def expert_sort(pick: torch.Tensor, n_experts: int, x: torch.Tensor, rank: torch.Tensor, counts: torch.Tensor,
                 place: torch.Tensor, xs: torch.Tensor, offsets: Optional[torch.Tensor] = None,
-                tile_group: Optional[torch.Tensor] = None) -> None:
+                tile_group: Optional[torch.Tensor] = None, in_w: Optional[torch.Tensor] = None) -> None:
     """The (token, choice) entries of ``pick`` [N, top] sorted by expert (stable): ``counts`` [experts] entries an
     expert, ``place`` [N * top] where each entry went, and the tokens' rows of ``x`` [N, H] copied to ``xs`` in that
     order, so that an expert's rows lie together.  With ``offsets`` [experts] and ``tile_group`` [tiles] every
     expert's run starts on a tile of ``GROUPED_TILE_ROWS`` rows (``xs`` then has tiles * that many rows, the rows
     between runs are left as they are), ``offsets`` says where, and ``tile_group`` names each tile's expert (-1 for
-    the spare tiles at the end): what :func:`gemm_tc_grouped` takes."""
+    the spare tiles at the end): what :func:`gemm_tc_grouped` takes.  ``in_w`` float32 [N, top]: an entry's copy of the row
+    is multiplied by its weight."""
     N, top = pick.shape
     H = x.shape[1]
     padded = offsets is not None
@@ -898,7 +904,7 @@ def expert_sort(pick: torch.Tensor, n_experts: int, x: torch.Tensor, rank: torch
             _need(tile_group, "tile groups", torch.int32), tile_group.numel(), _stream()), "mv_expert_tiles")
     _check(_fn("core", "mv_expert_gather")(
         pick.data_ptr(), rank.data_ptr(), counts.data_ptr(), offsets.data_ptr() if padded else None,
-        _need(x, "expert_sort rows", None, (N, H)), _dt(x), N, top, H,
+        _need(x, "expert_sort rows", None, (N, H)), _dt(x), _need(in_w, "input weights", torch.float32, (N, top), True), N, top, H,
         _need(place, "places", torch.int32, (N * top,)), _need(xs, "sorted rows", x.dtype, (rows, H)), _stream()),
         "mv_expert_gather")
     account(N * (1 + top) * H * x.element_size())
@@ -940,19 +946,19 @@ def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_gr
     return out
 
 
-def expert_combine(ys: torch.Tensor, place: torch.Tensor, pick_w: torch.Tensor, shared: Optional[torch.Tensor],
+def expert_combine(ys: torch.Tensor, place: torch.Tensor, pick_w: Optional[torch.Tensor], shared: Optional[torch.Tensor],
                    gate: Optional[torch.Tensor], out: torch.Tensor, accumulate: bool) -> torch.Tensor:
     """out[n] (+)= sum_k pick_w[n, k] * ys[place[n * top + k]] (+ gate[n] * shared[n]), float32: the chosen experts'
-    results gathered back in the order of the choices.  ``gate`` [N, 1] may be a column of a wider matrix.  ``ys``
+    results gathered back in the order of the choices (``pick_w`` None: every one counts as it is).  ``gate`` [N, 1] may be a column of a wider matrix.  ``ys``
     has at least N * top rows (more where the experts' runs are padded)."""
     N, H = out.shape
-    top = pick_w.shape[1]
+    top = place.numel() // N
     if ys.shape[0] < N * top:
         raise KernelError(f"expert_combine: {ys.shape[0]} result rows for {N * top} entries")
     gp, ldg = _cols(gate, "shared gate", N, 1) if gate is not None else (None, 0)
     _check(_fn("core", "mv_expert_combine")(
         _need(ys, "expert results", torch.float32, (None, H)), _need(place, "places", torch.int32, (N * top,)),
-        _need(pick_w, "pick weights", torch.float32, (N, top)), _need(shared, "shared result", torch.float32, (N, H), True),
+        _need(pick_w, "pick weights", torch.float32, (N, top), True), _need(shared, "shared result", torch.float32, (N, H), True),
         gp, ldg, _need(out, "combine out", torch.float32), N, top, H, int(bool(accumulate)), _stream()), "mv_expert_combine")
     account(N * H * 4 * (top + 2 + (1 if shared is not None else 0)))
     return out
@@ -1041,12 +1047,15 @@ def _check_kv_wide(pool: torch.Tensor, nkv: int, page_size: int, dk: int, dv: in
 def qkv_prepare_wide(proj: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float,
                      rot_dims: int, inv_freq: Optional[torch.Tensor], positions, seq_of, page_table,
                      pool: torch.Tensor, page_size: int, q_out: torch.Tensor, nh: int, nkv: int, dk: int,
-                     dv: int, *, per_head: bool = False, amplitude: float = 1.0) -> torch.Tensor:
+                     dv: int, *, per_head: bool = False, amplitude: float = 1.0,
+                     q_temp: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """From a row [q | k | v | ...] of a fused projection (float32, any row stride): root-mean-square norm over
     the whole of q and the whole of k (weights wq [nh * dk], wk [nkv * dk]; None: no norm), or with
     ``per_head`` over every head by itself (weights wq, wk [dk], shared by the heads); rotation of the
     first ``rot_dims`` elements of every head (element i with i + rot_dims / 2, angle pos * inv_freq[i], cos and
-    sin times ``amplitude``), q out in the model's dtype, k and v into the token's row of its page."""
+    sin times ``amplitude``), q out in the model's dtype, k and v into the token's row of its page.  ``q_temp`` (coef, every): q is
+    multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p.  ``nkv`` 0: the rows hold q alone, and the cache
+    is left as it is (a layer that reads another layer's keys and values)."""
     N = q_out.shape[0]
     need = nh * dk + nkv * (dk + dv)
     if (not proj.is_cuda or proj.dtype != torch.float32 or proj.dim() != 2 or proj.shape[0] != N or proj.shape[1] < need
@@ -1055,7 +1064,10 @@ def qkv_prepare_wide(proj: torch.Tensor, wq: Optional[torch.Tensor], wk: Optiona
                           f"{tuple(proj.shape)}")
     if rot_dims % 2 or not 0 <= rot_dims <= dk:
         raise KernelError(f"qkv_prepare_wide: {rot_dims} rotated elements in heads of {dk}")
-    _check_kv_wide(pool, nkv, page_size, dk, dv, "qkv_prepare_wide")
+    if nkv:
+        _check_kv_wide(pool, nkv, page_size, dk, dv, "qkv_prepare_wide")
+    if q_temp is not None and not q_temp[1] > 0:
+        raise KernelError(f"qkv_prepare_wide: the query temperature steps every {q_temp[1]} positions")
     if pool.dtype != q_out.dtype:
         raise KernelError(f"qkv_prepare_wide: cache is {pool.dtype} but q is {q_out.dtype}")
     _guard("core", "attention_sink", proj.device, n_pages=pool.shape[0])
@@ -1066,7 +1078,7 @@ def qkv_prepare_wide(proj: torch.Tensor, wq: Optional[torch.Tensor], wk: Optiona
         _need(positions, "positions", torch.int32), _need(seq_of, "seq_of", torch.int32),
         _need(page_table, "page table", torch.int32), page_table.shape[1], page_size, _need(pool, "cache pool"),
         pool.stride(0), _need(q_out, "q out", None, (N, nh * dk)), _dt(q_out), N, nh, nkv, dk, dv, int(bool(per_head)),
-        float(amplitude), _stream()), "mv_qkv_prepare_wide")
+        float(amplitude), *(map(float, q_temp) if q_temp is not None else (0.0, 0.0)), _stream()), "mv_qkv_prepare_wide")
     account(N * need * 4 + N * (nh * dk + nkv * (dk + dv)) * q_out.element_size())
     return q_out
 
@@ -1075,7 +1087,8 @@ def attention_sink(q: torch.Tensor, pool: torch.Tensor, page_size: int, page_tab
                    out: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, scale: float, *, softcap: float = 0.0,
                    window: int = 0, keep_first: int = 0, sinks: Optional[torch.Tensor] = None,
                    gate: Optional[torch.Tensor] = None, head_tile: int = 0, chunk: int = 0,
-                   distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, values_in_keys: bool = False,
+                   distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None,
+                   distance_table: Optional[torch.Tensor] = None, values_in_keys: bool = False,
                    gate_wide: bool = False, out_all: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal softmax attention of every token of the step over its sequence's cache (which already holds the
     step's own keys), keys of size dk and values of size dv.  ``softcap`` c > 0: s <- c tanh(s / c).  ``window``
@@ -1084,7 +1097,8 @@ def attention_sink(q: torch.Tensor, pool: torch.Tensor, page_size: int, page_tab
     multiplied by sigmoid(gate).  ``chunk`` c > 0 (instead of a window): query i reads key j <= i only if
     i // c == j // c.  ``head_tile``: how many query heads of a kv head share a block and its loads
     (1, 2 or 4; 0: the kernel chooses by the step's size).  ``distance_bias`` (r1, r2), float32 [nh] each:
-    r1_h ln(1 + r2_h (i - j)) is taken off the score.  ``values_in_keys``: the values are the first dv elements of
+    r1_h ln(1 + r2_h (i - j)) is taken off the (capped) score.  ``distance_table`` float32 [nh, L] (instead):
+    its entry [h, min(i - j, L - 1)] is added to the (capped) score.  ``values_in_keys``: the values are the first dv elements of
     the key rows and a page holds key rows only.  ``gate_wide``: ``gate`` is [N, nh * dv], one logit an element.
     ``out_all``: float32 [N, nh, nkv, dv]; every head's weights are applied to the values of every kv head and
     written there (``out`` is then left alone): what :func:`mix_heads` needs."""
@@ -1098,6 +1112,7 @@ def attention_sink(q: torch.Tensor, pool: torch.Tensor, page_size: int, page_tab
         raise KernelError(f"attention: q {q.dtype}, cache {pool.dtype}, out {out.dtype} must agree")
     gp, ldg = _cols(gate, "attention gate", N, nh * dv if gate_wide else nh) if gate is not None else (None, 0)
     r1, r2 = _bias_pair(distance_bias, nh, values_in_keys, dk, dv)
+    dist, dist_len = _distance_table(distance_table, distance_bias, nh)
     _guard("core", "attention_sink", q.device, n_pages=pool.shape[0])
     _check(_fn("core", "mv_attention_sink")(
         _need(q, "q", None, (N, nh * dk)), _need(pool, "cache pool"), pool.stride(0),
@@ -1106,7 +1121,7 @@ def attention_sink(q: torch.Tensor, pool: torch.Tensor, page_size: int, page_tab
         _need(sinks, "sinks", torch.float32, (nh,), True), gp, ldg,
         _need(out, "attention out", None, (N, nh * dv), out_all is not None),
         _dt(q), N, nh, nkv, dk, dv, float(scale), float(softcap), int(window), int(keep_first), int(head_tile),
-        int(chunk), r1, r2, int(bool(values_in_keys)), int(bool(gate_wide)),
+        int(chunk), r1, r2, dist, dist_len, int(bool(values_in_keys)), int(bool(gate_wide)),
         _need(out_all, "attention out of all kv heads", torch.float32, (N, nh, nkv, dv), True), _stream()), "mv_attention_sink")
     return out if out_all is None else out_all
 
@@ -1118,6 +1133,14 @@ def _bias_pair(distance_bias, nh: int, values_in_keys: bool, dk: int, dv: int):
         return None, None
     r1, r2 = distance_bias
     return _need(r1, "distance bias r1", torch.float32, (nh,)), _need(r2, "distance bias r2", torch.float32, (nh,))
+
+
+def _distance_table(table: Optional[torch.Tensor], distance_bias, nh: int):
+    if table is None:
+        return None, 0
+    if distance_bias is not None:
+        raise KernelError("attention: a distance bias is either two numbers a head or a table")
+    return _need(table, "distance table", torch.float32, (nh, None)), table.shape[1]
 
 
 def mix_heads(o_all: torch.Tensor, talk: torch.Tensor, out: torch.Tensor, nh: int, nkv: int, dv: int) -> torch.Tensor:
@@ -1147,6 +1170,7 @@ def attention_sink_prefill(q: torch.Tensor, pool: torch.Tensor, page_size: int, 
                            softcap: float = 0.0, window: int = 0, keep_first: int = 0,
                            sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                            chunk: int = 0, distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None,
+                           distance_table: Optional[torch.Tensor] = None,
                            values_in_keys: bool = False, gate_wide: bool = False,
                            out_all: Optional[torch.Tensor] = None, split_weights: bool = False) -> torch.Tensor:
     """:func:`attention_sink` for a step with many query tokens, on the tensor cores (bfloat16, key and value
@@ -1164,6 +1188,7 @@ def attention_sink_prefill(q: torch.Tensor, pool: torch.Tensor, page_size: int, 
         raise KernelError(f"attention: q {q.dtype}, cache {pool.dtype}, out {out.dtype} must agree")
     gp, ldg = _cols(gate, "attention gate", N, nh * dv if gate_wide else nh) if gate is not None else (None, 0)
     r1, r2 = _bias_pair(distance_bias, nh, values_in_keys, dk, dv)
+    dist, dist_len = _distance_table(distance_table, distance_bias, nh)
     _guard("bf16", "attention_sink_prefill", q.device, n_pages=pool.shape[0])
     _check(_fn("bf16", "mv_attention_sink_prefill")(
         _need(q, "q", None, (N, nh * dk)), _need(pool, "cache pool"), pool.stride(0),
@@ -1172,7 +1197,7 @@ def attention_sink_prefill(q: torch.Tensor, pool: torch.Tensor, page_size: int, 
         _need(sinks, "sinks", torch.float32, (nh,), True), gp, ldg,
         _need(out, "attention out", None, (N, nh * dv), out_all is not None),
         N, n_seqs, nh, nkv, dk, dv, float(scale), float(softcap), int(window), int(keep_first), int(chunk), r1, r2,
-        int(bool(values_in_keys)), int(bool(gate_wide)),
+        dist, dist_len, int(bool(values_in_keys)), int(bool(gate_wide)),
         _need(out_all, "attention out of all kv heads", torch.float32, (N, nh, nkv, dv), True), int(bool(split_weights)),
         _stream()), "mv_attention_sink_prefill")
     return out if out_all is None else out_all
@@ -1226,11 +1251,11 @@ LATENT_MAX_ROT = 512
 def latent_prepare(proj: torch.Tensor, q0: int, c0: int, w_c: torch.Tensor, eps: float, inv_freq: Optional[torch.Tensor],
                    positions, seq_of, page_table, pool: torch.Tensor, page_size: int, qa: torch.Tensor, nh: int, dim: int,
                    rot: int, rank: int, rot_dims: Optional[int] = None, cq0: int = 0, w_q: Optional[torch.Tensor] = None,
-                   cq: Optional[torch.Tensor] = None) -> None:
+                   cq: Optional[torch.Tensor] = None, amplitude: float = 1.0) -> None:
     """From float32 rows of a fused projection (q at column ``q0``: per head [dim | rot]; the latent at column ``c0``:
     [rank | rot]): the latent's first ``rank`` numbers over their root mean square times ``w_c``, its last ``rot`` and
     every head's last ``rot`` of q rotated (their first ``rot_dims``, all by default: element i with i + rot_dims / 2,
-    angle pos * inv_freq[i]; the others pass unchanged); the row [rank + rot]
+    angle pos * inv_freq[i], cos and sin times ``amplitude``; the others pass unchanged); the row [rank + rot]
     goes into the token's place of its page, the rotated parts of q into the last ``rot`` columns of ``qa``
     [N, nh, rank + rot] (float32; None: the queries are prepared elsewhere, and ``q0`` is not looked at).  ``cq``
     [N, q_rank] in the pool's dtype: the queries' own latent, from column ``cq0``, over its root mean square times
@@ -1255,7 +1280,7 @@ def latent_prepare(proj: torch.Tensor, q0: int, c0: int, w_c: torch.Tensor, eps:
         _need(positions, "positions", torch.int32), _need(seq_of, "seq_of", torch.int32),
         _need(page_table, "page table", torch.int32), page_table.shape[1], int(page_size), pool.data_ptr(), pool.stride(0),
         _dt(pool), _need(qa, "absorbed q", torch.float32, (N, nh, rank + rot), True), N, nh, dim, rot, rank, rot_dims,
-        int(cq0), cq.shape[1] if cq is not None else 0,
+        float(amplitude), int(cq0), cq.shape[1] if cq is not None else 0,
         _need(w_q, "query latent norm weight", torch.float32, (cq.shape[1],)) if cq is not None else None,
         _need(cq, "query latent", pool.dtype, (N, None), True), _stream()), "mv_latent_prepare")
     account(N * ((nh * rot * 8 if qa is not None else 0) + (rank + rot + (cq.shape[1] if cq is not None else 0)) * (4 + pool.element_size())))
@@ -1263,13 +1288,13 @@ def latent_prepare(proj: torch.Tensor, q0: int, c0: int, w_c: torch.Tensor, eps:
 
 def head_product(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, nh: int, n_in: int, n_out: int, *,
                  transposed: bool = False, gate: Optional[torch.Tensor] = None, rot: int = 0, rot_dims: int = 0,
-                 inv_freq: Optional[torch.Tensor] = None, positions=None) -> torch.Tensor:
+                 inv_freq: Optional[torch.Tensor] = None, positions=None, amplitude: float = 1.0) -> torch.Tensor:
     """One small matrix per head: y[n, h, :n_out] = W_h x[n, h, :n_in] with ``w`` [nh * n_out, n_in], or with
     ``transposed`` W_h^T x with ``w`` [nh * n_in, n_out].  ``x`` float32 [N, nh, >= n_in] and ``y`` [N, nh, >= n_out]
     (float32 or the model's dtype) may be views with any row and head strides.  ``gate``: float32 logits
     [N, nh * n_out], or [N, nh] for one a head (a column slice is fine); the result is multiplied by sigmoid(gate).
     ``rot`` > 0: the ``rot`` elements of x after its ``n_in`` are turned (their first ``rot_dims``: i with
-    i + rot_dims / 2, angle positions * inv_freq[i]; the others pass unchanged) and written after y's ``n_out``
+    i + rot_dims / 2, angle positions * inv_freq[i], cos and sin times ``amplitude``; the others pass unchanged) and written after y's ``n_out``
     (float32)."""
     N = x.shape[0]
     if rot and (y.dtype != torch.float32 or rot_dims % 2 or not 0 <= rot_dims <= rot):
@@ -1285,7 +1310,7 @@ def head_product(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, nh: int, n_i
     _check(_fn("core", "mv_head_product")(
         x.data_ptr(), x.stride(0), x.stride(1), _need(w, "head matrices", None, (rows, cols)), _dt(w), int(bool(transposed)),
         gp, ldg, int(per_head), y.data_ptr(), _dt(y), y.stride(0), y.stride(1), N, nh, int(n_in), int(n_out), int(rot),
-        int(rot_dims), _need(inv_freq, "inv_freq", torch.float32, (rot_dims // 2,)) if rot_dims else None,
+        int(rot_dims), float(amplitude), _need(inv_freq, "inv_freq", torch.float32, (rot_dims // 2,)) if rot_dims else None,
         _need(positions, "positions", torch.int32) if rot else None, _stream()), "mv_head_product")
     account(w.numel() * w.element_size() + N * nh * (n_in * 4 + n_out * y.element_size()), 2 * N * nh * n_in * n_out)
     return y
@@ -1383,9 +1408,10 @@ def latent_prefill_fits(dim: int, rot: int, dv: int, rank: int) -> bool:
 
 
 def latent_query(proj: torch.Tensor, q0: int, inv_freq: Optional[torch.Tensor], positions, q: torch.Tensor, nh: int,
-                 dim: int, rot: int, rot_dims: int) -> torch.Tensor:
+                 dim: int, rot: int, rot_dims: int, amplitude: float = 1.0) -> torch.Tensor:
     """``q`` [N, nh, dim + rot] (bfloat16) from float32 rows of a projection (the queries from column ``q0``), the first
-    ``rot_dims`` of every head's last ``rot`` elements turned (i with i + rot_dims / 2, angle pos * inv_freq[i])."""
+    ``rot_dims`` of every head's last ``rot`` elements turned (i with i + rot_dims / 2, angle pos * inv_freq[i], cos and sin times
+    ``amplitude``)."""
     N = q.shape[0]
     if (not proj.is_cuda or proj.dtype != torch.float32 or proj.dim() != 2 or proj.shape[0] != N or proj.stride(1) != 1
             or q0 < 0 or q0 + nh * (dim + rot) > proj.shape[1] or rot_dims % 2 or not 0 <= rot_dims <= rot):
@@ -1394,7 +1420,7 @@ def latent_query(proj: torch.Tensor, q0: int, inv_freq: Optional[torch.Tensor], 
     _check(_fn("bf16", "mv_latent_query")(
         proj.data_ptr(), proj.stride(0), int(q0), _need(inv_freq, "inv_freq", torch.float32, (rot_dims // 2,), rot_dims == 0),
         _need(positions, "positions", torch.int32), _need(q, "q", torch.bfloat16, (N, nh, dim + rot)), N, nh, dim, rot,
-        int(rot_dims), _stream()), "mv_latent_query")
+        int(rot_dims), float(amplitude), _stream()), "mv_latent_query")
     account(N * nh * (dim + rot) * 6)
     return q
 
@@ -1496,8 +1522,17 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Te
 SWIGLU_GROUP = 16
 
 
-def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int = 0) -> torch.Tensor:
-    """out[n, f] = silu(gate) * up.  ``group`` 0: gate and up are the two halves
+GLU_SILU, GLU_GELU = "silu", "gelu_tanh"
+
+
+def _glu_act(act: str) -> int:
+    if act not in (GLU_SILU, GLU_GELU):
+        raise KernelError(f"gated activation {act!r}; known: {GLU_SILU}, {GLU_GELU}")
+    return int(act == GLU_GELU)
+
+
+def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int = 0, act: str = GLU_SILU) -> torch.Tensor:
+    """out[n, f] = silu(gate) * up, or with ``act`` "gelu_tanh" gelu(gate) * up (the tanh form).  ``group`` 0: gate and up are the two halves
     of a row of ``gu``; 16: they alternate in groups of 16 columns."""
     N, F2 = gu.shape
     F = F2 // 2
@@ -1505,7 +1540,7 @@ def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int = 0) -> torch.Tensor:
         raise KernelError(f"swiglu: width {F} is not a multiple of the group size {group}")
     _check(_fn("core", "mv_swiglu")(
         _need(gu, "swiglu in", torch.float32), _need(out, "swiglu out", None, (N, F)), _dt(out), N, F, int(group),
-        _stream()), "mv_swiglu")
+        _glu_act(act), _stream()), "mv_swiglu")
     account(_nbytes(gu, out))
     return out
 
@@ -1572,10 +1607,35 @@ def glu_limits(widths_and_limits, alpha: float, device) -> torch.Tensor:
     return torch.cat(rows + [torch.tensor([float(alpha)], dtype=torch.float32)]).to(device)
 
 
-def _glu_mode(N: int, bias: Optional[torch.Tensor], limits: Optional[torch.Tensor]):
+@dataclass
+class ExpertWeights:
+    """Weights a row and an expert for a product over experts' gate and up rows laid end to end: ``dense`` float32
+    [rows, >= n_experts], the router's; an expert has ``ff`` features (a multiple of 16).  Features after the last
+    expert's (a shared one's) take 1."""
+    dense: torch.Tensor
+    n_experts: int
+    ff: int
+
+
+def _expert_weight_args(ew: Optional[ExpertWeights], M: int):
+    if ew is None:
+        return (None, 0, 0, 0)
+    if ew.ff % SWIGLU_GROUP or ew.dense.dim() != 2 or ew.dense.shape[0] != M or ew.dense.shape[1] < ew.n_experts:
+        raise KernelError(f"gemm: weights {tuple(ew.dense.shape)} for {M} rows and {ew.n_experts} experts of {ew.ff} features")
+    return (_need(ew.dense, "expert weights", torch.float32), ew.dense.shape[1], ew.ff // SWIGLU_GROUP, ew.n_experts)
+
+
+def _glu_mode(N: int, bias: Optional[torch.Tensor], limits: Optional[torch.Tensor], act: str = GLU_SILU,
+              weights: Optional[ExpertWeights] = None):
     """(mode, row stride of the output, what goes in the bias's place) of a product whose epilogue gates."""
+    if (limits is not None) + bool(_glu_act(act)) + (weights is not None) > 1:
+        raise KernelError("gemm: one of the clamped activation, gelu and experts' weights an epilogue")
+    if weights is not None:
+        if bias is not None:
+            raise KernelError("gemm: an epilogue with experts' weights takes no bias")
+        return 6, N // 2, None
     if limits is None:
-        return 3, N // 2, bias
+        return (5 if _glu_act(act) else 3), N // 2, bias
     if bias is not None:
         raise KernelError("gemm: the clamped activation's epilogue takes no bias")
     return 4, N // 2, limits
@@ -1588,7 +1648,7 @@ def gemm_small_m_tile_rows(N: int, mode: int) -> int:
 def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
                  accumulate: bool = False, swiglu: bool = False, scale: Optional[NormLink] = None,
                  emit: Optional[NormLink] = None, ahead: Optional[tuple] = None,
-                 limits: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 limits: Optional[torch.Tensor] = None, act: str = GLU_SILU) -> torch.Tensor:
     """out = x @ w.T for at most 64 rows of x, bfloat16 operands: the
     weight-streaming tensor-core kernel of the decode step.  ``scale`` / ``emit``: the
     two ends of a :class:`NormLink`.  ``ahead``: (address, bytes) of what the step's next
@@ -1605,7 +1665,7 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: O
     if swiglu:
         if N % 32:
             raise KernelError(f"gemm_small_m: the SwiGLU epilogue needs rows in groups of 32, got {N}")
-        mode, ldo, bias = _glu_mode(N, bias, limits)
+        mode, ldo, bias = _glu_mode(N, bias, limits, act)
         _need(out, "gemm out", torch.bfloat16, (M, N // 2))
     elif accumulate:
         mode = 2
@@ -1815,13 +1875,15 @@ def gemm_tc_pair_takes(M: int, N: int) -> bool:
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
             accumulate: bool = False, swiglu: bool = False, pair: Optional[bool] = None,
             scale: Optional[NormLink] = None, emit: Optional[NormLink] = None,
-            limits: Optional[torch.Tensor] = None) -> torch.Tensor:
+            limits: Optional[torch.Tensor] = None, act: str = GLU_SILU,
+            weights: Optional[ExpertWeights] = None) -> torch.Tensor:
     """out = x @ w.T, bfloat16 operands, on the tcgen05 tensor cores (TMA
     loads, accumulator in tensor memory): the matrix product of prefill.
     ``pair``: True: the kernel in which two multiprocessors share a 256 x 256 tile, False: the
     one-multiprocessor kernels, None: by shape (``gemm_tc_pair_takes``).  ``scale`` / ``emit``: the two
     ends of a :class:`NormLink`; every kernel here applies a scale, only the pair kernel emits (N in
-    steps of 32)."""
+    steps of 32).  With ``swiglu``: ``act`` "gelu_tanh" takes gelu instead of silu; ``weights``: gate and up rows of experts
+    end to end, multiplied by a weight a row and an expert before the activation."""
     M, K = x.shape
     N, K2 = w.shape
     if K != K2:
@@ -1834,7 +1896,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
     if swiglu:
         if N % 32:
             raise KernelError(f"gemm_tc: the SwiGLU epilogue needs rows in groups of 32, got {N}")
-        mode, ldo, bias = _glu_mode(N, bias, limits)
+        mode, ldo, bias = _glu_mode(N, bias, limits, act, weights)
         _need(out, "gemm out", torch.bfloat16, (M, N // 2))
     elif accumulate:
         mode = 2
@@ -1853,7 +1915,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
         link = _link_args(x, M, N, K, mode, scale, emit, -(-N // 256))
         _check(_fn("bf16", "mv_gemm_tc_pair")(
             _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N + (mode == 4),), True),
-            out.data_ptr(), mode, M, N, K, ldo, *link, _error_flag(x.device).data_ptr(), _stream()), "mv_gemm_tc_pair")
+            out.data_ptr(), mode, M, N, K, ldo, *link, *_expert_weight_args(weights, M), _error_flag(x.device).data_ptr(),
+            _stream()), "mv_gemm_tc_pair")
         _account_gemm(x, w, out, accumulate)
         return out
     if emit is not None:
@@ -1862,7 +1925,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
     entry = "mv_gemm_tc"
     _check(_fn("bf16", entry)(
         _need(x, "gemm x"), _need(w, "gemm w"), _need(bias, "gemm bias", torch.float32, (N + (mode == 4),), True),
-        out.data_ptr(), mode, M, N, K, ldo, *link[:5], _error_flag(x.device).data_ptr(), _stream()), entry)
+        out.data_ptr(), mode, M, N, K, ldo, *link[:5], *_expert_weight_args(weights, M), _error_flag(x.device).data_ptr(),
+        _stream()), entry)
     _account_gemm(x, w, out, accumulate)
     return out
 
@@ -1870,7 +1934,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Option
 def gemm_tc_swap(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
                  accumulate: bool = False, swiglu: bool = False, scale: Optional[NormLink] = None,
                  emit: Optional[NormLink] = None, ahead: Optional[tuple] = None,
-                 limits: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 limits: Optional[torch.Tensor] = None, act: str = GLU_SILU) -> torch.Tensor:
     """out = x @ w.T on the tcgen05 tensor cores with the operands' roles swapped (rows of w
     on the MMA's M side, up to 256 tokens a tile on its N side): a TMA pipeline that streams w
     once, K cut over the blocks of a cluster.  Same contract as ``gemm_small_m``, for any number of
@@ -1887,7 +1951,7 @@ def gemm_tc_swap(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: O
     if swiglu:
         if N % 32:
             raise KernelError(f"gemm_tc_swap: the SwiGLU epilogue needs rows in groups of 32, got {N}")
-        mode, ldo, bias = _glu_mode(N, bias, limits)
+        mode, ldo, bias = _glu_mode(N, bias, limits, act)
         _need(out, "gemm out", torch.bfloat16, (M, N // 2))
     elif accumulate:
         mode = 2

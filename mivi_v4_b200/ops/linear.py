@@ -228,20 +228,27 @@ def end_norms_carried(n_rows: int) -> bool:
 
 
 def linear_swiglu(x: torch.Tensor, w_grouped: torch.Tensor, out: torch.Tensor, *,
-                  scale: Optional[K.NormLink] = None, limits: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  scale: Optional[K.NormLink] = None, limits: Optional[torch.Tensor] = None,
+                  act: str = K.GLU_SILU, weights: Optional[K.ExpertWeights] = None) -> torch.Tensor:
     """out = silu(gate) * up where [gate | up] = x @ w_grouped.T and the rows of
     ``w_grouped`` alternate in groups of 16 (gate rows, then the up rows of the
     same features): the activation runs in the product's epilogue, so gate and
-    up never go to memory.  ``limits`` (``kernels.glu_limits``): the clamped gated activation instead.  Needs
-    ``tensor_core_ok``."""
+    up never go to memory.  ``limits`` (``kernels.glu_limits``): the clamped gated activation instead; ``act``
+    "gelu_tanh": gelu instead of silu; ``weights`` (steps of more than 64 rows): a weight a row and an expert on gate and
+    up.  Needs ``tensor_core_ok``."""
+    if weights is not None:
+        if _order is not None:
+            _order.next_after(w_grouped)
+        return K.gemm_tc(x, w_grouped, out, swiglu=True, scale=scale, weights=weights)
     if x.shape[0] <= K.SMALL_M_MAX:
         fn = _small_m(x.shape[0])
-        return fn(x, w_grouped, out, swiglu=True, scale=scale, limits=limits, **_ahead(w_grouped, fn))
+        return fn(x, w_grouped, out, swiglu=True, scale=scale, limits=limits, act=act, **_ahead(w_grouped, fn))
     if swap_takes(x.shape[0], w_grouped):
-        return K.gemm_tc_swap(x, w_grouped, out, swiglu=True, scale=scale, limits=limits, **_ahead(w_grouped, K.gemm_tc_swap))
+        return K.gemm_tc_swap(x, w_grouped, out, swiglu=True, scale=scale, limits=limits, act=act,
+                              **_ahead(w_grouped, K.gemm_tc_swap))
     if _order is not None:
         _order.next_after(w_grouped)
-    return K.gemm_tc(x, w_grouped, out, swiglu=True, scale=scale, limits=limits)
+    return K.gemm_tc(x, w_grouped, out, swiglu=True, scale=scale, limits=limits, act=act)
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,

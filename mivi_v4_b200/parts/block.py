@@ -248,19 +248,46 @@ class PreNormScaledBlock(Part):
 class PostNormBlock(Part):
     """x += norm1(mixer(x)); then, if the layer has a feed-forward, x += norm2(feed_forward(x)): the norms sit on
     the sublayers' OUTPUTS and the sublayers read the stream itself (rounded to the model's dtype where that is
-    narrower).  The norms are root-mean-square norms.  One kernel per sublayer adds a mixer's branches (a mixer
-    with ``forward_sum`` gives them apart, with their factors), norms the sum, adds it to the float32 stream and
+    narrower).  The norms are root-mean-square norms or layer norms.  With ``scaled`` each normed result is multiplied
+    element by element by a learned vector (``scale1`` the mixer's, ``scale2`` the feed-forward's), which is put into the
+    norm's weight and bias once, in float32, when the weights are loaded.  One kernel per sublayer adds a mixer's branches
+    (a mixer with ``forward_sum`` gives them apart, with their factors), norms the sum, adds it to the float32 stream and
     writes the rounded rows that the next sublayer multiplies."""
 
     nested_roles = {"mixer": "mixer", "mixer_norm": "norm", "ffn": "feed_forward", "ffn_norm": "norm"}
 
-    def __init__(self, mixer, mixer_norm, ffn=None, ffn_norm=None):
+    def __init__(self, mixer, mixer_norm, ffn=None, ffn_norm=None, scaled: bool = False):
         if (ffn is None) != (ffn_norm is None):
             raise ValueError("a feed-forward and its norm come together or not at all")
         for norm in (mixer_norm, ffn_norm):
-            if norm is not None and not isinstance(norm, RMSNorm):
-                raise ValueError("the norms of a postnorm block are rmsnorm parts")
+            if norm is not None and not isinstance(norm, (RMSNorm, LayerNorm)):
+                raise ValueError("the norms of a postnorm block are rmsnorm or layernorm parts")
         self.mixer, self.mixer_norm, self.ffn, self.ffn_norm = mixer, mixer_norm, ffn, ffn_norm
+        self.scaled = bool(scaled)
+        self.joins = {}
+
+    def param_specs(self):
+        from .spec import ParamSpec
+        if not self.scaled:
+            return {}
+        specs = {"scale1": ParamSpec((self.mixer_norm.dim,), "vector", "norm")}
+        if self.ffn is not None:
+            specs["scale2"] = ParamSpec((self.ffn_norm.dim,), "vector", "norm")
+        return specs
+
+    def load_named(self, named) -> None:
+        super().load_named(named)
+        # what a sublayer's joining kernel multiplies and adds: the norm's weight and (a layer norm's) bias, times the vector
+        for norm, vec in ((self.mixer_norm, "scale1"), (self.ffn_norm, "scale2")):
+            if norm is None:
+                continue
+            w, b = norm.weight, getattr(norm, "bias", None)
+            if b is None and isinstance(norm, LayerNorm):
+                b = torch.zeros_like(w)
+            if self.scaled:
+                v = getattr(self, vec).float()
+                w, b = (w * v).contiguous(), None if b is None else (b * v).contiguous()
+            self.joins[norm] = (w, b)
 
     def nested(self):
         parts = {"mixer": self.mixer, "mixer_norm": self.mixer_norm, "ffn": self.ffn, "ffn_norm": self.ffn_norm}
@@ -292,7 +319,8 @@ class PostNormBlock(Part):
         if len(rest) > 1:
             raise ValueError("at most two branches are summed in the norm's kernel")
         y2, s2 = rest[0] if rest else (None, 1.0)
-        K.rmsnorm_add_sum(y1, norm.weight, norm.eps, resid, s1=s1, y2=y2, s2=s2, rounded=rounded)
+        w, b = self.joins[norm]
+        K.norm_add_sum(y1, w, norm.eps, resid, bias=b, s1=s1, y2=y2, s2=s2, rounded=rounded)
 
     def forward(self, resid, step, view, after=None) -> None:
         N, H = resid.shape

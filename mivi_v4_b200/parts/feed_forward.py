@@ -15,7 +15,7 @@ from .spec import ParamSpec
 @register("feed_forward", "swiglu")
 class SwiGLU(Part):
     """x + (silu(g W1^T) * (g W3^T)) W2^T without biases
-    (crates/mivi-model/src/ffn.rs:56-108).  W1 and W3 are merged at load time
+    (crates/mivi-model/src/ffn.rs:56-108); with ``act`` "gelu_tanh" gelu in its tanh form instead of silu.  W1 and W3 are merged at load time
     so that one product yields gate and up: in alternating groups of 16 rows
     (16 of W1, then the 16 of W3 for the same features) when the width allows,
     which lets the tensor-core kernels apply the activation in their
@@ -23,8 +23,10 @@ class SwiGLU(Part):
 
     overwrites = True            # forward(..., accumulate=False) writes its result instead of adding it
 
-    def __init__(self, hidden: int, ff: int):
-        self.hidden, self.ff = int(hidden), int(ff)
+    def __init__(self, hidden: int, ff: int, act: str = "silu"):
+        if act not in (K.GLU_SILU, K.GLU_GELU):
+            raise ValueError(f"feed-forward activation {act!r}; known: {K.GLU_SILU}, {K.GLU_GELU}")
+        self.hidden, self.ff, self.act = int(hidden), int(ff), act
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         H, F = self.hidden, self.ff
@@ -51,11 +53,11 @@ class SwiGLU(Part):
         N = g.shape[0]
         h = self.scratch(step, "ffh", (N, self.ff), step.dtype)
         if self.group and tensor_core_ok(g, self.w13):
-            linear_swiglu(g, self.w13, h, scale=scale)
+            linear_swiglu(g, self.w13, h, scale=scale, act=self.act)
         else:
             gu = self.scratch(step, "proj", (N, 2 * self.ff), torch.float32)
             linear(g, self.w13, gu, scale=scale)
-            K.swiglu(gu, h, self.group)
+            K.swiglu(gu, h, self.group, self.act)
         linear(h, self.w2, resid, accumulate=accumulate, emit=emit)
 
 
@@ -104,12 +106,14 @@ class RoutedExperts(Part):
     is the input itself times the weight.  The entries form ``n_groups`` equal
     groups of neighbours, a group's score is the sum of its two largest scores, and only experts of the
     ``keep_groups`` best groups can be chosen; the ``top`` largest scores among them are chosen and weigh their
-    experts by s / (sum of the chosen s + 1e-20).  With ``shared_ff`` > 0 a shared expert of that width runs for
+    experts by s / (sum of the chosen s + 1e-20), or without ``renormalize`` by s itself.  With ``weight_on`` "input" the
+    weight multiplies the expert's INPUT, expert(w h), and its output counts as it is.  With ``shared_ff`` > 0 a shared expert of that width runs for
     every token and is added times sigmoid(w_sg . h), or as it is without ``shared_gate``.
 
     All experts' gate and up matrices are laid end to end (the shared expert's last), so that one product yields
     every expert's pre-activations; the gated activation is multiplied by the router's weight before it is
-    rounded (zero where an expert was not chosen: nothing is computed there), and one product with the down
+    rounded (or gate and up are, before the activation, where the input carries the weight; zero where an expert was not
+    chosen: nothing is computed there), and one product with the down
     matrices side by side sums the chosen experts.  Long bfloat16 steps instead sort the (token, choice) entries by
     expert on the device and run grouped products over the sorted rows, so every expert multiplies its own tokens
     only.  No decision is taken on the host."""
@@ -121,7 +125,8 @@ class RoutedExperts(Part):
     def __init__(self, hidden: int, n_experts: int, ff: int, top: int, n_groups: int = 1, keep_groups: int = 1,
                  shared_ff: int = 0, score: str = "sigmoid", correction: bool = False, out_scale: float = 1.0,
                  n_identity: int = 0, router_bias: bool = False, shared_gate: bool = True, act: str = "silu",
-                 limit: float = 0.0, shared_limit: float = 0.0, alpha: float = 1.702):
+                 limit: float = 0.0, shared_limit: float = 0.0, alpha: float = 1.702, renormalize: bool = True,
+                 weight_on: str = "output"):
         routed = int(n_experts) + int(n_identity)
         if n_experts < 1 or n_identity < 0 or routed > K.MAX_EXPERTS or n_groups < 1 or routed % n_groups:
             raise ValueError(f"{routed} routed entries do not form {n_groups} equal groups (at most {K.MAX_EXPERTS})")
@@ -138,6 +143,9 @@ class RoutedExperts(Part):
         self.I, self.routed = int(n_identity), routed
         self.has_router_bias, self.shared_gate = bool(router_bias), bool(shared_gate) and self.shared_ff > 0
         self.clamped, self.limit, self.shared_limit, self.alpha = act == "clamped", float(limit), float(shared_limit), float(alpha)
+        if weight_on not in ("output", "input") or (weight_on == "input" and self.clamped):
+            raise ValueError(f"router weights on the experts' {weight_on!r} (output or input) with activation {act!r}")
+        self.renormalize, self.on_input = bool(renormalize), weight_on == "input"
         self.side, self._side_at = None, None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -236,21 +244,25 @@ class RoutedExperts(Part):
         pick_w = self.scratch(step, "pick_w", (N, self.top), torch.float32)
         K.route(z[:, :cols], dense, pick, pick_w, self.routed, self.n_groups, self.keep, self.top, self.shared_gate,
                 mode=self.SCORES[self.score], correction=self.correction, out_scale=self.out_scale, n_identity=I,
-                bias=self.router_bias)
+                bias=self.router_bias, renormalize=self.renormalize)
         if self._sorted_ok(g, step, N):
             return self._forward_sorted(g, resid, step, accumulate, dense, pick, pick_w)
         h = self.scratch(step, "ffh", (N, F), step.dtype)
         if (N >= self.GATED_IN_PRODUCT_FROM and self.group and (self.shared_group or not self.shared_ff)
-                and tensor_core_ok(g, self.w_gu)):
+                and tensor_core_ok(g, self.w_gu) and not (self.on_input and self.shared_gate)):
             # long steps: gate and up never reach memory; the weights go on the rounded activations
-            linear_swiglu(g, self.w_gu, h, limits=self.all_limits)
-            K.scale_expert_columns(h, dense, E, self.ff, self.shared_ff, extra_cols=I, shared_gate=self.shared_gate)
+            # (on the input: on gate and up inside the product)
+            if self.on_input:
+                linear_swiglu(g, self.w_gu, h, weights=K.ExpertWeights(dense, E, self.ff))
+            else:
+                linear_swiglu(g, self.w_gu, h, limits=self.all_limits)
+                K.scale_expert_columns(h, dense, E, self.ff, self.shared_ff, extra_cols=I, shared_gate=self.shared_gate)
         else:
             gu = self.scratch(step, "proj", (N, 2 * F), torch.float32)
             linear(g, self.w_gu, gu)
             clamp = dict(limit=self.limit, shared_limit=self.shared_limit, alpha=self.alpha) if self.clamped else {}
             K.routed_glu(gu, dense, h, E, self.ff, self.shared_ff, self.group, self.shared_group, extra_cols=I,
-                         shared_gate=self.shared_gate, **clamp)
+                         shared_gate=self.shared_gate, on_input=self.on_input, **clamp)
         linear(h, self.w_down, resid, accumulate=accumulate)
         if I:
             K.identity_experts(g, dense, E + sg, I, resid)
@@ -266,7 +278,7 @@ class RoutedExperts(Part):
         tile_group = self.scratch(step, "tile_group", (tiles,), torch.int32)
         place = self.scratch(step, "place", (N * top,), torch.int32)
         xs = self.scratch(step, "sorted", (rows, H), g.dtype)
-        K.expert_sort(pick, E, g, rank, counts, place, xs, offsets, tile_group)
+        K.expert_sort(pick, E, g, rank, counts, place, xs, offsets, tile_group, in_w=pick_w if self.on_input else None)
         hs = self.scratch(step, "sorted_h", (rows, ff), step.dtype)
         K.gemm_tc_grouped(xs, self.w_gu, hs, tile_group, 2 * ff, H, row_step=2 * ff, swiglu=True, active_rows=N * top,
                           limits=self.expert_limits)
@@ -288,4 +300,4 @@ class RoutedExperts(Part):
             shared = self.scratch(step, "shared_y", (N, H), torch.float32)
             linear(hsh, self._shared_down[0], shared)
         # the shared expert's gate, where it has one, is the last column of the router's dense weights
-        K.expert_combine(ys, place, pick_w, shared, dense[:, E:E + 1] if self.shared_gate else None, resid, accumulate)
+        K.expert_combine(ys, place, None if self.on_input else pick_w, shared, dense[:, E:E + 1] if self.shared_gate else None, resid, accumulate)

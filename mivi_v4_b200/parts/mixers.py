@@ -2,7 +2,8 @@
 from __future__ import annotations
 
 import math
-from typing import Dict, Optional
+from fractions import Fraction
+from typing import Dict, Optional, Tuple
 
 import torch
 
@@ -295,6 +296,30 @@ class LightningAttention(Part):
         linear(y, self.w_o, resid, accumulate=True)
 
 
+def distance_table(rel: torch.Tensor, reach) -> torch.Tensor:
+    """A bias by distance bucket, ``rel`` [rows, heads], as a table [heads, L] by distance: column n belongs to a key n >= 0
+    tokens back, and the last column to every longer distance.  Row n serves the nearest rows // 2 distances (call that
+    number h); from there on distance n takes row h + floor(ln(n / h) / ln(reach / h) * (rows - h)), at most the last one:
+    rows for ever longer stretches, the last one from about ``reach`` on.  The edges are compared as whole numbers,
+    (n / h)^(rows - h) with (reach / h)^k, so that a distance that lies on one falls on its far side on every machine."""
+    rows = rel.shape[0]
+    h, far = rows // 2, Fraction(reach)
+    if h < 1 or not far > h:
+        raise ValueError(f"a bias table of {rows} rows that reaches {reach} tokens: it needs at least 2 rows, and a reach "
+                         f"beyond the rows // 2 nearest distances")
+    steps = rows - h
+    index = list(range(h))
+    n, k = h, 0
+    while True:
+        while k + 1 < steps and Fraction(n) ** steps * h ** (k + 1) >= far ** (k + 1) * h ** steps:
+            k += 1
+        index.append(h + k)
+        if k + 1 == steps:
+            break
+        n += 1
+    return rel[torch.tensor(index, device=rel.device)].T.contiguous()
+
+
 @register("mixer", "sink_attention")
 class SinkAttention(Part):
     """Grouped-query softmax attention over the cache with keys of size ``key_dim`` and values of size
@@ -320,7 +345,13 @@ class SinkAttention(Part):
     the scores (``r1``, ``r2`` [heads]).  ``sink`` "zero": the sink's score is 0 for every head and there is no
     tensor (the denominator gains 1).  ``gated`` "element": the gate is one projection of the layer's input per
     element of the concatenated heads.  ``split_weights``: steps of many tokens carry 16 instead of 8 bits of a
-    softmax weight's mantissa into the value product."""
+    softmax weight's mantissa into the value product.
+
+    ``proj_bias``: q, k and v have biases (``q.b``, ``k.b``, ``v.b``), added in the projection.  ``q_temp`` (coef, every): q
+    is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p.  ``bias_max`` D > 0: a learned number a head and
+    distance bucket (``rel`` [B, heads], B rows as the checkpoint has them or ``bias_rows``) is added to the scaled and capped
+    score, the buckets as ``distance_table`` lays them out.  ``shared_kv``: the layer has no keys and values of its own and
+    reads those that another layer's cache holds (its schedule entry says which)."""
 
     nested_roles = {"position": "position"}
     overwrites = True            # forward(..., accumulate=False) writes its result instead of adding it
@@ -329,7 +360,9 @@ class SinkAttention(Part):
                  position, softcap: float = 0.0, window: int = 0, keep_first: int = 0,
                  qk_norm_eps: Optional[float] = None, sink=True, gated=True,
                  norm_per_head: bool = False, chunk: int = 0, talk: bool = False, conv: int = 0,
-                 values_are_keys: bool = False, distance_bias: bool = False, split_weights: bool = False):
+                 values_are_keys: bool = False, distance_bias: bool = False, split_weights: bool = False,
+                 proj_bias: bool = False, q_temp: Optional[Tuple[float, float]] = None, bias_max: float = 0,
+                 bias_rows: Optional[int] = None, shared_kv: bool = False):
         if n_kv_heads < 1 or n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads are not a multiple of {n_kv_heads} kv heads")
         if not (1 <= key_dim <= K.MAX_HEAD_DIM and 1 <= value_dim <= K.MAX_HEAD_DIM):
@@ -344,6 +377,13 @@ class SinkAttention(Part):
         self.norm_per_head, self.chunk = bool(norm_per_head), int(chunk)
         self.talk, self.conv, self.values_are_keys = bool(talk), int(conv), bool(values_are_keys)
         self.distance_bias, self.split_weights = bool(distance_bias), bool(split_weights)
+        self.proj_bias, self.shared_kv = bool(proj_bias), bool(shared_kv)
+        self.q_temp = None if q_temp is None else (float(q_temp[0]), float(q_temp[1]))
+        self.bias_max, self.bias_rows = bias_max or 0, None if bias_rows is None else int(bias_rows)
+        if self.shared_kv and (self.conv or self.talk):
+            raise ValueError("a layer that reads another layer's keys and values has no convolution and no mixed heads")
+        if self.bias_max and self.distance_bias:
+            raise ValueError("a distance bias is either two numbers a head or a table")
         if self.values_are_keys and self.dv > self.dk:
             raise ValueError(f"values of {self.dv} cannot be the first elements of keys of {self.dk}")
         if not 0 <= self.conv <= K.MAX_CONV_K:
@@ -365,13 +405,21 @@ class SinkAttention(Part):
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         H, nh, nkv, dk, dv = self.hidden, self.nh, self.nkv, self.dk, self.dv
-        specs = {"q": ParamSpec((nh * dk, H)), "k": ParamSpec((nkv * dk, H))}
-        if not self.values_are_keys:
-            specs["v"] = ParamSpec((nkv * dv, H))
+        rows = {"q": nh * dk}
+        if not self.shared_kv:
+            rows["k"] = nkv * dk
+            if not self.values_are_keys:
+                rows["v"] = nkv * dv
+        specs = {n: ParamSpec((r, H)) for n, r in rows.items()}
+        if self.proj_bias:
+            specs.update({n + ".b": ParamSpec((r,), "vector", "bias") for n, r in rows.items()})
         specs["o"] = ParamSpec((H, nh * dv))
         if self.qk_norm_eps is not None:
             specs["q.norm"] = ParamSpec((dk if self.norm_per_head else nh * dk,), "vector", "norm")
-            specs["k.norm"] = ParamSpec((dk if self.norm_per_head else nkv * dk,), "vector", "norm")
+            if not self.shared_kv:
+                specs["k.norm"] = ParamSpec((dk if self.norm_per_head else nkv * dk,), "vector", "norm")
+        if self.bias_max:
+            specs["rel"] = ParamSpec((self.bias_rows, nh), "vector", "norm")
         if self.sink is True:
             specs["sink"] = ParamSpec((nh,), "vector", "bias")
         if self.gated:
@@ -387,7 +435,13 @@ class SinkAttention(Part):
         return specs
 
     def load(self, t) -> None:
-        self.w_qkvg = _fuse_rows([t["q"], t["k"]] + ([] if self.values_are_keys else [t["v"]]) + ([t["g"]] if self.gated else []))
+        names = [n for n in ("q", "k", "v") if n in t]
+        self.w_qkvg = _fuse_rows([t[n] for n in names] + ([t["g"]] if self.gated else []))
+        self.b_qkvg = None
+        if self.proj_bias:
+            b = torch.cat([t[n + ".b"].float() for n in names])
+            self.b_qkvg = torch.nn.functional.pad(b, (0, self.w_qkvg.shape[0] - b.shape[0])).contiguous()
+        self.by_distance = distance_table(t["rel"].float(), self.bias_max) if self.bias_max else None
         self.w_o = t["o"]
         self.q_norm, self.k_norm, self.sinks = t.get("q.norm"), t.get("k.norm"), t.get("sink")
         if self.sink == "zero":
@@ -407,8 +461,11 @@ class SinkAttention(Part):
         conv_state = None
         if self.conv > 1:
             view, conv_state = view[0], view[1].state
+        if view.writable == self.shared_kv:
+            raise RuntimeError("a shared_kv attention layer must read another layer's cache, and only it may")
+        own_kv = 0 if self.shared_kv else nkv
         proj = self.scratch(step, "proj", (N, self.w_qkvg.shape[0]), torch.float32)
-        linear(u, self.w_qkvg, proj)
+        linear(u, self.w_qkvg, proj, bias=self.b_qkvg)
         rot = self.position.rotary(u.device) if self.rot_dims else None
         q = self.scratch(step, "q", (N, nh * dk), step.dtype)
         rows = proj
@@ -418,15 +475,15 @@ class SinkAttention(Part):
                           step.n_seqs, one_each=step.is_decode)
         K.qkv_prepare_wide(rows, self.q_norm, self.k_norm, self.qk_norm_eps or 0.0, self.rot_dims,
                            rot[0] if rot is not None else None, step.positions, step.seq_of, view.page_table,
-                           view.pool, view.page_size, q, nh, nkv, dk, 0 if self.values_are_keys else dv,
-                           per_head=self.norm_per_head,
+                           view.pool, view.page_size, q, nh, own_kv, dk, 0 if self.values_are_keys else dv,
+                           per_head=self.norm_per_head, q_temp=self.q_temp,
                            amplitude=float(getattr(self.position, "amplitude", lambda: 1.0)()) if self.rot_dims else 1.0)
         o = self.scratch(step, "mix", (N, nh * dv), step.dtype)
-        g0 = nh * dk + nkv * dk + (0 if self.values_are_keys else nkv * dv)
+        g0 = nh * dk + own_kv * (dk + (0 if self.values_are_keys else dv))
         wide = self.gated == "element"
         extras = dict(softcap=self.softcap, window=self.window, keep_first=self.keep_first, sinks=self.sinks,
                       gate=proj[:, g0:g0 + (nh * dv if wide else nh)] if self.gated else None, chunk=self.chunk,
-                      distance_bias=self.bias, values_in_keys=self.values_are_keys, gate_wide=wide,
+                      distance_bias=self.bias, distance_table=self.by_distance, values_in_keys=self.values_are_keys, gate_wide=wide,
                       out_all=self.scratch(step, "o_all", (N, nh, nkv, dv), torch.float32) if self.talk else None)
         # few query tokens, or many sequences with a token or two each: every query token on its own
         few = N <= K.DECODE_ATTENTION_MAX_TOKENS or step.max_len <= K.DECODE_ATTENTION_MAX_QUERIES
@@ -654,7 +711,10 @@ class LatentAttention(Part):
     denominator; with ``gated`` the concatenated heads are multiplied by sigmoid(W_g h), element by element ("element",
     or True) or head by head ("head": W_g has a row a head); then W_o.  With ``q_rank`` the queries come through a latent
     of their own: q = W_uq c_q, c_q = W_dq h over its root mean square times a weight.  The position
-    part turns the first ``position.head_dim`` of the ``rot_dim`` elements, element i with i + head_dim / 2.
+    part turns the first ``position.head_dim`` of the ``rot_dim`` elements, element i with i + head_dim / 2; where it
+    pairs neighbours (2i, 2i + 1) instead, the rows of the matrices that make rotated elements are put in the other order
+    when they are loaded, which no score can tell (queries and keys are turned alike).  A position part with an
+    ``amplitude()`` has its cos and sin multiplied by it.
 
     Only [c | r] is cached, one row a token for all heads.  W_uk is folded into the query
     (qa = [W_uk^T q_unrotated | q_rotated]) and W_uv applied to the weighted sum of the cached c, so keys and values
@@ -676,8 +736,8 @@ class LatentAttention(Part):
         self.q_rank = int(q_rank)
         self.rot_dims = 0
         if isinstance(position, Rope):
-            if position.style != "half_split" or position.head_dim > self.rd:
-                raise ValueError("the rotation pairs element i with i + dims / 2 over at most the rotated size")
+            if position.head_dim > self.rd:
+                raise ValueError(f"{position.head_dim} elements turn, of a rotated size of {self.rd}")
             self.rot_dims = position.head_dim
         elif position.rotary("cpu") is not None:
             raise ValueError("a rotation that is not a Rope part cannot say how many elements it turns")
@@ -701,6 +761,14 @@ class LatentAttention(Part):
         return specs
 
     def load(self, t) -> None:
+        if self.rot_dims and self.position.style == "interleaved":
+            t = dict(t)
+            first = torch.arange(self.rot_dims, device=t["dkv"].device)
+            order = torch.cat([first[0::2], first[1::2], torch.arange(self.rot_dims, self.rd, device=first.device)])
+            up = "uq" if self.q_rank else "q"
+            heads = t[up].view(self.nh, self.dim + self.rd, -1)
+            t[up] = torch.cat([heads[:, :self.dim], heads[:, self.dim:][:, order]], dim=1).reshape(t[up].shape).contiguous()
+            t["dkv"] = torch.cat([t["dkv"][:self.rank], t["dkv"][self.rank:][order]]).contiguous()
         self.w_in = _fuse_rows([t["dq" if self.q_rank else "q"], t["dkv"]] + ([t["g"]] if self.gated else []))
         self.c_norm, self.sinks, self.w_o = t["dkv.norm"], t.get("sink"), t["o"]
         self.q_norm, self.w_uq = t.get("dq.norm"), t.get("uq")
@@ -739,6 +807,7 @@ class LatentAttention(Part):
             self.side = proj[:, self._side_at[0]:self._side_at[0] + self._side_at[1]]
         rot = self.position.rotary(u.device) if self.rot_dims else None
         inv_freq = rot[0] if rot is not None else None
+        amplitude = float(self.position.amplitude()) if self.rot_dims else 1.0
         gate = proj[:, g0:g0 + self.gate_rows] if self.gated else None
         y = self.scratch(step, "mix", (N, nh * dv), step.dtype)
         rows = self._seen_rows(step) if step.max_len >= self.LONG_STEP else 0
@@ -757,12 +826,12 @@ class LatentAttention(Part):
             qa = self.scratch(step, "qa", (N, nh, rank + rd), torch.float32)
         K.latent_prepare(proj, 0, c0, self.c_norm, self.eps, inv_freq, step.positions, step.seq_of, view.page_table,
                          view.pool, view.page_size, None if self.q_rank else qa, nh, dim, rd, rank, self.rot_dims,
-                         w_q=self.q_norm, cq=cq)
+                         w_q=self.q_norm, cq=cq, amplitude=amplitude)
         if self.q_rank:
             linear(cq, self.w_uq, queries)
         if long:
             q = self.scratch(step, "q", (N, nh, dim + rd), torch.bfloat16)
-            K.latent_query(queries, 0, inv_freq, step.positions, q, nh, dim, rd, self.rot_dims)
+            K.latent_query(queries, 0, inv_freq, step.positions, q, nh, dim, rd, self.rot_dims, amplitude)
             c = self.scratch(step, "c", (rows, rank), torch.bfloat16)
             r = self.scratch(step, "r", (rows, rd), torch.bfloat16)
             K.latent_gather(view.pool, view.page_size, view.page_table, step.cu, step.starts, step.n_seqs, self.window, c, r)
@@ -776,7 +845,8 @@ class LatentAttention(Part):
             linear(y, self.w_o, resid, accumulate=accumulate)
             return
         # (queries that latent_prepare did not see are turned here)
-        turn = dict(rot=rd, rot_dims=self.rot_dims, inv_freq=inv_freq, positions=step.positions) if self.q_rank and rd else {}
+        turn = dict(rot=rd, rot_dims=self.rot_dims, inv_freq=inv_freq, positions=step.positions,
+                    amplitude=amplitude) if self.q_rank and rd else {}
         K.head_product(queries[:, :nh * (dim + rd)].unflatten(1, (nh, dim + rd)), w_uk, qa, nh, dim, rank, transposed=True, **turn)
         o_lat = self.scratch(step, "o_lat", (N, nh, rank), torch.float32)
         # few query tokens with many keys each: the keys in shares.  The number of shares follows from what the page

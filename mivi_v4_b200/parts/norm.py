@@ -46,10 +46,11 @@ class RMSNorm(Part):
 class LayerNorm(Part):
     """y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * weight (+ bias, with ``bias``) over the last
     dimension, in float32.  It is not carried by the products around it (it has no ``link``): it always runs as
-    a kernel."""
+    a kernel.  ``gain``: a constant factor on the result (a final norm whose logits are scaled), put into weight and bias
+    once, in float32, when they are loaded."""
 
-    def __init__(self, dim: int, eps: float, bias: bool = False):
-        self.dim, self.eps, self.has_bias = int(dim), float(eps), bool(bias)
+    def __init__(self, dim: int, eps: float, bias: bool = False, gain: float = 1.0):
+        self.dim, self.eps, self.has_bias, self.gain = int(dim), float(eps), bool(bias), float(gain)
         self.weight: Optional[torch.Tensor] = None
         self.bias: Optional[torch.Tensor] = None
 
@@ -58,6 +59,10 @@ class LayerNorm(Part):
         if self.has_bias:
             specs["bias"] = ParamSpec((self.dim,), "vector", "bias")
         return specs
+
+    def load(self, t) -> None:
+        self.weight = (t["weight"].float() * self.gain).contiguous()
+        self.bias = (t["bias"].float() * self.gain).contiguous() if self.has_bias else None
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         return K.layernorm(x, self.weight, self.eps, out, rows, bias=self.bias)

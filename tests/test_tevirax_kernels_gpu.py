@@ -359,7 +359,7 @@ def test_gate_before_the_grouped_norm_and_the_post_norm_sum():
     for second in (None, y2):
         r = dev(resid)
         rounded = torch.empty(N, C, dtype=torch.bfloat16, device=DEV)
-        k.rmsnorm_add_sum(dev(y), dev(w), 1e-5, r, s1=0.7, y2=None if second is None else dev(second), s2=1.3, rounded=rounded)
+        k.norm_add_sum(dev(y), dev(w), 1e-5, r, s1=0.7, y2=None if second is None else dev(second), s2=1.3, rounded=rounded)
         total = 0.7 * y + (1.3 * second if second is not None else 0)
         close(r, resid + P.rms_norm(total, w, 1e-5), 1e-5, "post-norm sum")
         assert torch.equal(rounded, r.to(torch.bfloat16))
