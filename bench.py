@@ -12,6 +12,7 @@ prefill, then generation timed without its first token).
     python bench.py --design puzorax [--stages ..]      (the Puzorax decoder beside the Tevirax decoder of equal sizes)
     python bench.py --design ropelix [--stages ..]      (the Ropelix decoder beside the Tevirax decoder of equal sizes)
     python bench.py --design redisun [--stages ..]      (the Redisun decoder beside the Puzorax decoder of equal sizes)
+    python bench.py --design mevulix [--stages ..]      (the Mevulix decoder beside the Redisun decoder of equal sizes)
     python bench.py --kernel NAME [--m .. --n .. --k ..] (one kernel alone, for timing and for profilers)
 
 One "step" is one decode step of the whole batch.  Prints ONE JSON line:
@@ -280,6 +281,22 @@ def redisun_config(width, layers, heads, kv_heads, ff, vocab):
                        for i in range(layers)]}
 
 
+def mevulix_config(width, layers, heads, kv_heads, ff, vocab):
+    """Two layers of latent attention with a query latent (the Redisun sizes), then a layer of grouped-query attention with
+    a bias by distance, and so on, every second attention layer reading the keys and values of the one before it; the
+    first layer's feed-forward is dense, the others are mixtures of 16 experts of an eighth of its width, 4 chosen, and a
+    shared one of the same width."""
+    latent = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256, "q_rank": width // 4, "scale": 96 ** -0.5,
+              "rot": {"dims": 32, "base": 1000000.0, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 50.0,
+           "q_temp": {"coef": 0.1, "every": 4096}, "bias_rows": 64, "bias_max": 1000}
+    moe = {"kind": "moe", "expert": {"ff": ff // 8}, "shared": {"ff": ff // 8}, "router": {"experts": 16, "top": 4}}
+    return {"architecture": "Mevulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [{"type": "attention" if i % 3 == 2 else "latent_attention",
+                        "mixer": (dict(att, kv_from=i - 3) if i % 6 == 5 else att) if i % 3 == 2 else latent,
+                        "mlp": {"kind": "dense", "ff": ff} if i == 0 else moe} for i in range(layers)]}
+
+
 def lfm2_like(width, layers, heads, kv_heads, ff, vocab):
     cfg = dict(BENCH_CONFIG)
     cfg.update(hidden_size=width, num_hidden_layers=layers, num_attention_heads=heads, num_key_value_heads=kv_heads,
@@ -291,17 +308,17 @@ def lfm2_like(width, layers, heads, kv_heads, ff, vocab):
 def run_design(args, warmup: int) -> int:
     """Prefill and decode throughput of a further design (--design) at the sizes of DESIGN_SIZES, each beside its
     closest neighbour in the library at equal sizes (Votavik beside LFM2, Tevirax beside Votavik, Puzorax and Ropelix beside
-    Tevirax, Redisun beside Puzorax), random weights,
+    Tevirax, Redisun beside Puzorax, Mevulix beside Redisun), random weights,
     bfloat16: one JSON line.  With --stages: where a step of the design's model (--size) goes, kernel by kernel."""
     import torch
     from mivi_v4_b200 import measure, random_model
     pk, pk_src = peaks()
     # the design that was asked for, beside its closest neighbour in the library at equal sizes
     design_cfg = {"votavik": votavik_config, "tevirax": tevirax_config, "puzorax": puzorax_config,
-                  "ropelix": ropelix_config, "redisun": redisun_config}[args.design]
+                  "ropelix": ropelix_config, "redisun": redisun_config, "mevulix": mevulix_config}[args.design]
     beside, beside_cfg = {"votavik": ("lfm2", lfm2_like), "tevirax": ("votavik", votavik_config),
                           "puzorax": ("tevirax", tevirax_config), "ropelix": ("tevirax", tevirax_config),
-                          "redisun": ("puzorax", puzorax_config)}[args.design]
+                          "redisun": ("puzorax", puzorax_config), "mevulix": ("redisun", redisun_config)}[args.design]
     if args.stages:
         model = random_model(design_cfg(*DESIGN_SIZES[args.size]), seed=0, dtype="bfloat16", device="cuda:0", on_device=True)
         lens = [args.tokens] if args.stages == "prefill" else [args.prompt_len] * args.batch
@@ -422,7 +439,7 @@ def main() -> int:
     ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS),
                     help="run one of the two further workloads instead of the default benchmark")
     ap.add_argument("--size", default="w2048", choices=sorted(DESIGN_SIZES), help="with --design --stages: which size")
-    ap.add_argument("--design", default=None, choices=["votavik", "tevirax", "puzorax", "ropelix", "redisun"],
+    ap.add_argument("--design", default=None, choices=["votavik", "tevirax", "puzorax", "ropelix", "redisun", "mevulix"],
                     help="measure a further design beside its closest neighbour in the library at equal sizes (Votavik beside LFM2, "
                          "Tevirax beside Votavik) instead of the default benchmark")
     ap.add_argument("--stages", default=None, choices=["decode", "prefill"],
