@@ -289,7 +289,7 @@ def mevulix_config(width, layers, heads, kv_heads, ff, vocab):
     latent = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256, "q_rank": width // 4, "scale": 96 ** -0.5,
               "rot": {"dims": 32, "base": 1000000.0, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
     att = {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 50.0,
-           "q_temp": {"coef": 0.1, "every": 4096}, "bias_rows": 64, "bias_max": 1000}
+           "q_temp": {"coef": 0.1, "every": 4096}, "bias_rows": 64, "bias_max": 256}
     moe = {"kind": "moe", "expert": {"ff": ff // 8}, "shared": {"ff": ff // 8}, "router": {"experts": 16, "top": 4}}
     return {"architecture": "Mevulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
             "layers": [{"type": "attention" if i % 3 == 2 else "latent_attention",

@@ -113,6 +113,8 @@ _SIGNATURES = {
         "mv_attention_prefill": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
         "mv_attention_sink_prefill": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I,
                                       _I, _I, _P, _P, _P, _I, _I, _I, _P, _I, _P],
+        "mv_attention_sink_decode": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P,
+                                     _P, _P],
         "mv_attention_decode_tc": [_P, _P, _Q, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _P, _P],
         "mv_attention_prefill_tc": [_P, _P, _Q, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
         "mv_latent_attention_decode": [_P, _P, _Q, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P, _P],
@@ -1155,6 +1157,57 @@ def mix_heads(o_all: torch.Tensor, talk: torch.Tensor, out: torch.Tensor, nh: in
         _need(o_all, "mix_heads input", torch.float32, (N, nh, nkv, dv)), _need(talk, "mix_heads talk", torch.float32, (nh, nh)),
         _need(out, "mix_heads out", None, (N, nh * dv)), _dt(out), N, nh, nkv, dv, _stream()), "mv_mix_heads")
     account(N * nh * dv * (4 * nkv + out.element_size()), 2 * N * nh * nh * dv)
+    return out
+
+
+SINK_DECODE_KEYS, SINK_DECODE_HEADS, SINK_DECODE_MAX_SPLITS = 64, 16, 32
+
+
+def attention_sink_decode_supported(dtype: torch.dtype, dk: int, dv: int) -> bool:
+    """What the tensor-core kernel for steps of few query tokens takes: bfloat16, key and value sizes that are multiples of
+    16 (up to 256)."""
+    return dtype == torch.bfloat16 and dk % 16 == 0 and dv % 16 == 0 and 16 <= dk <= MAX_HEAD_DIM and 16 <= dv <= MAX_HEAD_DIM
+
+
+def attention_sink_decode_splits(n_tokens: int, nh: int, nkv: int, longest: int, sm_count: int) -> int:
+    """Into how many shares of the keys :func:`attention_sink_decode` cuts a step of ``n_tokens`` query tokens: three blocks
+    a multiprocessor, no share under a tile of keys."""
+    blocks = max(1, n_tokens * nkv * -(-(nh // nkv) // SINK_DECODE_HEADS))
+    return int(max(1, min(3 * sm_count // blocks, longest // SINK_DECODE_KEYS, SINK_DECODE_MAX_SPLITS)))
+
+
+def attention_sink_decode(q: torch.Tensor, pool: torch.Tensor, page_size: int, page_table, positions, seq_of,
+                          out: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, scale: float, *, softcap: float = 0.0,
+                          window: int = 0, chunk: int = 0, sinks: Optional[torch.Tensor] = None,
+                          distance_table: Optional[torch.Tensor] = None, splits: int = 1,
+                          part: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> torch.Tensor:
+    """:func:`attention_sink` for steps of few query tokens on the tensor cores (``attention_sink_decode_supported``): the
+    query heads of a kv head are the rows of both products; a softmax weight enters the value product as two bfloat16
+    numbers (16 bits of its mantissa).  ``splits`` > 1: the keys of every token are cut into that many shares, one block
+    each, and a second kernel puts the shares together; ``part`` = (float32 [N, nh, splits, dv], float32 [N, nh, splits, 2])
+    is their scratch."""
+    N, splits = q.shape[0], int(splits)
+    if not attention_sink_decode_supported(q.dtype, dk, dv):
+        raise KernelError(f"attention_sink_decode: needs bfloat16 and key and value sizes 16..{MAX_HEAD_DIM} in steps of 16, "
+                          f"got {q.dtype}, {dk}, {dv}")
+    if nkv < 1 or nh % nkv:
+        raise KernelError(f"attention: {nh} heads are not a multiple of {nkv} kv heads")
+    _check_kv_wide(pool, nkv, page_size, dk, dv, "attention_sink_decode")
+    if q.dtype != pool.dtype or out.dtype != q.dtype:
+        raise KernelError(f"attention: q {q.dtype}, cache {pool.dtype}, out {out.dtype} must agree")
+    if not 1 <= splits <= SINK_DECODE_MAX_SPLITS or (splits > 1 and part is None):
+        raise KernelError(f"attention_sink_decode: {splits} shares of the keys (1..{SINK_DECODE_MAX_SPLITS}) need their scratch")
+    dist, dist_len = _distance_table(distance_table, None, nh)
+    _guard("bf16", "attention_sink_decode", q.device, n_pages=pool.shape[0])
+    _check(_fn("bf16", "mv_attention_sink_decode")(
+        _need(q, "q", None, (N, nh * dk)), _need(pool, "cache pool"), pool.stride(0),
+        _need(page_table, "page table", torch.int32), page_table.shape[1], page_size,
+        _need(positions, "positions", torch.int32), _need(seq_of, "seq_of", torch.int32),
+        _need(sinks, "sinks", torch.float32, (nh,), True), dist, dist_len, _need(out, "attention out", None, (N, nh * dv)),
+        N, nh, nkv, dk, dv, float(scale), float(softcap), int(window), int(chunk), splits,
+        _need(part[0], "shares", torch.float32, (N, nh, splits, dv)) if splits > 1 else None,
+        _need(part[1], "shares' sums", torch.float32, (N, nh, splits, 2)) if splits > 1 else None, _stream()),
+        "mv_attention_sink_decode")
     return out
 
 

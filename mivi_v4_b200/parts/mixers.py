@@ -380,6 +380,8 @@ class SinkAttention(Part):
         self.proj_bias, self.shared_kv = bool(proj_bias), bool(shared_kv)
         self.q_temp = None if q_temp is None else (float(q_temp[0]), float(q_temp[1]))
         self.bias_max, self.bias_rows = bias_max or 0, None if bias_rows is None else int(bias_rows)
+        # which layers the tensor-core kernel for steps of few tokens serves
+        self.decode_tc = not (self.gated or self.talk or self.values_are_keys or self.distance_bias or self.keep_first)
         if self.shared_kv and (self.conv or self.talk):
             raise ValueError("a layer that reads another layer's keys and values has no convolution and no mixed heads")
         if self.bias_max and self.distance_bias:
@@ -490,6 +492,20 @@ class SinkAttention(Part):
         if not few and K.attention_sink_prefill_supported(step.dtype, dk, dv):
             K.attention_sink_prefill(q, view.pool, view.page_size, view.page_table, step.cu, step.starts, o,
                                      step.n_seqs, nh, nkv, dk, dv, self.scale, split_weights=self.split_weights, **extras)
+        elif self.decode_tc and K.attention_sink_decode_supported(step.dtype, dk, dv):
+            # few query tokens: a kv head's query heads as the rows of both products, the keys in shares.  The number of
+            # shares follows from what the page table can hold, not from the lengths of the moment, so that a recorded step
+            # stays right as they grow.
+            longest = view.page_table.shape[1] * view.page_size
+            longest = min(longest, self.window or longest, self.chunk or longest)
+            splits = K.attention_sink_decode_splits(N, nh, nkv, longest, K.n_sms())
+            part = None
+            if splits > 1:
+                part = (self.scratch(step, "part_o", (N, nh, splits, dv), torch.float32),
+                        self.scratch(step, "part_ml", (N, nh, splits, 2), torch.float32))
+            K.attention_sink_decode(q, view.pool, view.page_size, view.page_table, step.positions, step.seq_of, o, nh, nkv,
+                                    dk, dv, self.scale, softcap=self.softcap, window=self.window, chunk=self.chunk,
+                                    sinks=self.sinks, distance_table=self.by_distance, splits=splits, part=part)
         else:
             K.attention_sink(q, view.pool, view.page_size, view.page_table, step.positions, step.seq_of, o, nh, nkv,
                              dk, dv, self.scale, **extras)

@@ -169,7 +169,8 @@ def _rounded(h, p, dtype):
 ATT = [(_m(6, 2, 32, 16, 0.4, 5.0, 0.8, 7, 40), 12, 16), (_m(1, 1, 8, 8, 1.0, 30.0, 0.5, 1, 64), 8, 64),
        (_m(3, 1, 11, 9, 0.5, 2.0, 1.5, 50, 20), 2, 8), (_m(4, 4, 16, 128, 0.7, 8.0, 0.3, 33, 2000), 31, 16),
        (_m(8, 1, 64, 48, 0.3, 20.0, 0.4, 64, 33), 9, 32), (_m(10, 5, 128, 64, 0.2, 9.0, 0.1, 100, 120), 16, 64),
-       (_m(2, 2, 250, 256, 0.2, 4.0, 0.6, 10, 7), 3, 16)]
+       (_m(2, 2, 250, 256, 0.2, 4.0, 0.6, 10, 7), 3, 16), (_m(12, 1, 48, 32, 0.4, 6.0, 0.2, 30, 90), 20, 16),
+       (_m(40, 2, 16, 16, 0.5, 5.0, 0.4, 25, 50), 6, 8), (_m(5, 5, 256, 256, 0.1, 9.0, 0.3, 12, 30), 10, 16)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -267,6 +268,61 @@ def test_a_distance_table_longer_than_shared_memory_holds_and_of_one_number(dtyp
             k.attention_sink_prefill(dev(q.reshape(T, -1), dtype), pool, ps, i32([rows[0]]), i32([0, T]), i32([0]), full, 1, H, G, dk, dv,
                                      0.2, softcap=4.0, distance_table=dev(table), split_weights=True)
             close(full[places], want, 1.5e-2, f"{L} distances on the tensor cores")
+            for splits in (1, 5):
+                part = (torch.empty(len(places), H, splits, dv, device=DEV), torch.empty(len(places), H, splits, 2, device=DEV))
+                k.attention_sink_decode(dev(q[places].reshape(-1, H * dk), dtype), pool, ps, i32([rows[0]]), i32(places), i32([0] * len(places)),
+                                        out, H, G, dk, dv, 0.2, softcap=4.0, distance_table=dev(table), splits=splits, part=part)
+                close(out, want, 1.5e-2, f"{L} distances, single tokens on the tensor cores, {splits} shares")
+
+
+@pytest.mark.parametrize("splits", [1, 2, 3, 7, 32])
+@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 64, 64), (9, 1, 32, 48), (20, 1, 16, 16), (8, 8, 128, 96), (3, 1, 80, 160), (2, 2, 240, 256)])
+def test_single_tokens_on_the_tensor_cores_windows_chunks_caps_sinks_and_shares(H, G, dk, dv, splits):
+    """Tokens at many places of two sequences, their keys in shares (some without any key), with a window or a chunked mask,
+    a key that stands out just inside and just outside, with and without a cap, a sink and a table."""
+    k = K()
+    T, ps = 230, 16
+    places, seqs = [0, 1, 15, 16, 17, 63, 64, 65, 99, 127, 128, 200, T - 1, 5, 77, 150], [0] * 13 + [1] * 3
+    key, v = rnd(2, T, G, dk).to(BF).double(), rnd(2, T, G, dv, seed=1).to(BF).double()
+    rows, n_pages = _pages([T, T], ps)
+    pool = torch.zeros(n_pages, G * ps * (dk + dv), dtype=BF, device=DEV)
+    for b in range(2):
+        for blk, page in enumerate(rows[b][:-(-T // ps)]):
+            n = min(ps, T - blk * ps)
+            pool[page, :G * ps * dk].view(G, ps, dk)[:, :n] = dev(key[b, blk * ps:blk * ps + n].permute(1, 0, 2), BF)
+            pool[page, G * ps * dk:].view(G, ps, dv)[:, :n] = dev(v[b, blk * ps:blk * ps + n].permute(1, 0, 2), BF)
+    if dk == dv:
+        pool = pool.view(n_pages, 2, G, ps, dk)
+    part = (torch.full((16, H, splits, dv), float("nan"), device=DEV), torch.full((16, H, splits, 2), float("nan"), device=DEV))
+    table, sink = rnd(H, 70, seed=4), rnd(H, seed=5)
+    for window, chunk, cap, with_sink, with_table in ((0, 0, 5.0, True, True), (64, 0, 0.0, True, False), (65, 0, 3.0, False, True),
+                                                      (0, 48, 0.0, False, False), (1, 0, 0.0, True, True), (0, 64, 9.0, True, False)):
+        q = rnd(16, H, dk, seed=2)
+        for n, (p, b) in enumerate(zip(places, seqs)):         # one key stands out: the first one seen, or the last one not seen
+            lo = max(0, p - window + 1) if window else (p - p % chunk if chunk else 0)
+            j = max(lo - n % 2, 0)
+            q[n] = q[n] + 3.0 * key[b, j].repeat_interleave(H // G, dim=0)
+        q = q.to(BF).double()
+        s = torch.einsum("nhd,nshd->nhs", q, torch.stack([key[b] for b in seqs]).repeat_interleave(H // G, dim=2)) * dk ** -0.5
+        s = cap * torch.tanh(s / cap) if cap else s
+        back = torch.tensor(places)[:, None] - torch.arange(T)[None, :]
+        if with_table:
+            s = s + table[:, back.clamp(0, 69)].permute(1, 0, 2)
+        gone = back < 0
+        if window:
+            gone = gone | (back >= window)
+        if chunk:
+            gone = gone | (torch.arange(T)[None, :] // chunk != torch.tensor(places)[:, None] // chunk)
+        s = s.masked_fill(gone[:, None, :], float("-inf"))
+        if with_sink:
+            s = torch.cat([s, sink[None, :, None].expand(16, H, 1)], -1)
+        w = torch.softmax(s, -1)[..., :T]
+        want = torch.einsum("nhs,nshd->nhd", w, torch.stack([v[b] for b in seqs]).repeat_interleave(H // G, dim=2)).reshape(16, -1)
+        out = torch.full((16, H * dv), float("nan"), dtype=BF, device=DEV)
+        k.attention_sink_decode(dev(q.reshape(16, -1), BF), pool, ps, i32(rows), i32(places), i32(seqs), out, H, G, dk, dv, dk ** -0.5,
+                                softcap=cap, window=window, chunk=chunk, sinks=dev(sink) if with_sink else None,
+                                distance_table=dev(table) if with_table else None, splits=splits, part=part)
+        close(out, want, 6e-3, f"window {window} chunk {chunk} cap {cap}")
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
