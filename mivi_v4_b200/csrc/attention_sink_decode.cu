@@ -46,6 +46,16 @@ __device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const void* 
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s) : "memory");
 }
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ unsigned bits(const __nv_bfloat162& v) { return *reinterpret_cast<const unsigned*>(&v); }
 
 struct Shape {
@@ -132,18 +142,14 @@ attention_sink_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
         for (int e = 0; e < 4; ++e) oacc[j][e] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;           // rows lane / 4 and lane / 4 + 8; l: this lane's share
     const int t4 = lane & 3, gq = lane >> 2;
-    const float inv_cap = S.cap > 0.f ? 1.0f / S.cap : 0.f;
+    const float cap_l = S.cap * LOG2E, scale_l = S.cap > 0.f ? 2.0f * LOG2E * S.scale / S.cap : S.scale * LOG2E;
     const float* d0 = dist ? dist + (size_t)(h0 + min(gq, heads - 1)) * S.dist_len : nullptr;
     const float* d1 = dist ? dist + (size_t)(h0 + min(gq + 8, heads - 1)) * S.dist_len : nullptr;
     const float far0 = dist ? d0[S.dist_len - 1] : 0.f, far1 = dist ? d1[S.dist_len - 1] : 0.f;
     auto score = [&](float x, float add) {                              // in units of log 2
-        x *= S.scale;
-        if (S.cap > 0.f) {
-            // tanh(x) = (1 - e^-2|x|) / (1 + e^-2|x|) with the fast exponential (within 1e-6 of the cap)
-            const float y = x * inv_cap, e2 = __expf(-2.0f * fabsf(y));
-            x = copysignf(S.cap * __fdividef(1.0f - e2, 1.0f + e2), y);
-        }
-        return (x + add) * LOG2E;
+        // a capped score: cap tanh(y), y = scale x / cap, as cap - 2 cap / (1 + e^(2y)) (within 1e-6 of the cap's size)
+        const float bias = add * LOG2E;
+        return S.cap > 0.f ? fmaf(-2.0f * cap_l, rcp(1.0f + ex2(x * scale_l)), cap_l + bias) : fmaf(x, scale_l, bias);
     };
     const __nv_bfloat16* q_at = qs + (lane & 15) * pk + (lane >> 4) * 8;
     const int k_at = ((lane & 7) + ((lane >> 4) & 1) * 8) * pk + ((lane >> 3) & 1) * 8;
@@ -191,21 +197,21 @@ attention_sink_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
         mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
         mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
         // (the first of the 16 keys is seen, so the maxima are finite)
-        const float mn0 = fmaxf(m0, mx0), c0 = exp2f(m0 - mn0);
+        const float mn0 = fmaxf(m0, mx0), c0 = ex2(m0 - mn0);
         m0 = mn0;
         float c1 = c0;
         if (!PACK) {
             mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
             mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
             const float mn1 = fmaxf(m1, mx1);
-            c1 = exp2f(m1 - mn1);
+            c1 = ex2(m1 - mn1);
             m1 = mn1;
         }
         unsigned ph[4], pl[4];
         float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
-            const float x = exp2f(s[t][0] - m0), y = exp2f(s[t][1] - m0);
+            const float x = ex2(s[t][0] - m0), y = ex2(s[t][1] - m0);
             sum0 += x + y;
             const __nv_bfloat162 hv = __floats2bfloat162_rn(x, y);
             const unsigned rest = bits(__floats2bfloat162_rn(x - __low2float(hv), y - __high2float(hv)));
@@ -214,7 +220,7 @@ attention_sink_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
                 ph[2 * t + 1] = rest;                                   // rows 8 to 15: the remainders
             } else {
                 pl[2 * t] = rest;
-                const float x1 = exp2f(s[t][2] - m1), y1 = exp2f(s[t][3] - m1);
+                const float x1 = ex2(s[t][2] - m1), y1 = ex2(s[t][3] - m1);
                 sum1 += x1 + y1;
                 const __nv_bfloat162 h1 = __floats2bfloat162_rn(x1, y1);
                 ph[2 * t + 1] = bits(h1);
@@ -265,8 +271,8 @@ attention_sink_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
         return M;
     };
     {
-        const float f0 = exp2f(m0 - top_of(gq));                        // (warp 0 has seen a key: the tops are finite)
-        const float f1 = PACK ? 0.f : exp2f(m1 - top_of(gq + 8));
+        const float f0 = ex2(m0 - top_of(gq));                        // (warp 0 has seen a key: the tops are finite)
+        const float f1 = PACK ? 0.f : ex2(m1 - top_of(gq + 8));
         float* o0 = os + (size_t)(warp * HT + gq) * op + 2 * t4;
         float* o1 = o0 + (size_t)8 * op;
 #pragma unroll
@@ -284,8 +290,8 @@ attention_sink_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
     __syncthreads();
     for (int r = warp; r < heads; r += NW) {
         const float M = top_of(r);
-        float L = with_sink ? exp2f(sinks[h0 + r] * LOG2E - M) : 0.f;
-        for (int k = 0; k < NW; ++k) L += l_s[k][r] * exp2f(m_s[k][r] - M);
+        float L = with_sink ? ex2(sinks[h0 + r] * LOG2E - M) : 0.f;
+        for (int k = 0; k < NW; ++k) L += l_s[k][r] * ex2(m_s[k][r] - M);
         const size_t row = (size_t)n * S.nh + h0 + r;
         const float inv = 1.0f / L;
         for (int c = lane; c < dv; c += 32) {

@@ -49,6 +49,21 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 __device__ __forceinline__ unsigned pack_rest(float lo, float hi, unsigned rounded) {
     return pack_bf16(lo - __uint_as_float(rounded << 16), hi - __uint_as_float(rounded & 0xffff0000u));
 }
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ void ldmatrix_x4(unsigned (&r)[4], const void* smem) {
+    const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
+}
 __device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const void* smem) {
     const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -70,22 +85,25 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
     __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(smem_raw);     // [2][KB][ldk]
     __nv_bfloat16* vs = ks + 2 * KB * ldk;                              // [2][KB][ldv]
 
-    int b = 0, tile = blockIdx.x;
+    // the heads of a tile one after the other, the last tiles (the longest walks) first
+    int b = 0, tile = gridDim.y - 1 - blockIdx.y;
     for (; b < B; ++b) {
         const int tiles = (cu[b + 1] - cu[b] + QT - 1) / QT;
         if (tile < tiles) break;
         tile -= tiles;
     }
     if (b >= B) return;
-    // with o_all the grid's y counts (head, kv head whose values are read)
-    const int h = o_all ? blockIdx.y / nkv : blockIdx.y, g = h / (nh / nkv);
-    const int vg = o_all ? blockIdx.y - h * nkv : g;
-    const float db1 = r1 ? r1[h] : 0.f, db2 = r1 ? r2[h] : 0.f;
+    // with o_all the grid's x counts (head, kv head whose values are read)
+    const int h = o_all ? blockIdx.x / nkv : blockIdx.x, g = h / (nh / nkv);
+    const int vg = o_all ? blockIdx.x - h * nkv : g;
+    // scores, maxima and biases are held in units of log 2: the weights are powers of two then
+    const float db1 = r1 ? r1[h] * LOG2E : 0.f, db2 = r1 ? r2[h] : 0.f;
     const float* by_dist = dist ? dist + (size_t)h * dist_len : nullptr;
-    const float beyond = dist ? by_dist[dist_len - 1] : 0.f;
+    const float beyond = dist ? by_dist[dist_len - 1] * LOG2E : 0.f;
+    const float dist_unit = dist_len <= DIST_SMEM ? 1.0f : LOG2E;
     if (dist && dist_len <= DIST_SMEM) {
         float* row = reinterpret_cast<float*>(vs + 2 * KB * ldv);       // (the loop's first barrier publishes it)
-        for (int i = threadIdx.x; i < dist_len; i += NWARPS * 32) row[i] = by_dist[i];
+        for (int i = threadIdx.x; i < dist_len; i += NWARPS * 32) row[i] = by_dist[i] * LOG2E;
         by_dist = row;
     }
     const int row0 = cu[b] + tile * QT;
@@ -124,9 +142,11 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
         for (int e = 0; e < 4; ++e) oacc[j][e] = 0.f;
     // the sink starts the running maximum and the denominator (its own term, exp(sink - max), is 1 now); the
     // denominator of a row is summed over the four lanes of its quad at the end, so one of them holds it
-    float m0 = sinks ? sinks[h] : -INFINITY, m1 = m0;
+    float m0 = sinks ? sinks[h] * LOG2E : -INFINITY, m1 = m0;
     float l0 = (sinks && t4 == 0) ? 1.f : 0.f, l1 = l0;
-    const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
+    // a capped score: cap tanh(y), y = scale s / cap, as cap - 2 cap / (1 + e^(2y)) (within 1e-6 of the cap's size, far
+    // below the rounding of the operands)
+    const float cap_l = cap * LOG2E, scale_l = cap > 0.f ? 2.0f * LOG2E * scale / cap : scale * LOG2E;
 
     // key blocks this tile walks: the blocks that hold kept first tokens and lie before the window's
     // blocks, then from the first query's window start to the last query's position
@@ -139,22 +159,22 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
     const int n_iter = n_kept + kb_end - kb_begin;
 
     auto load_block = [&](int kb, int buf) {
-        const int kchunks = dk >> 3, vchunks = dv >> 3;
-        for (int idx = threadIdx.x; idx < KB * (kchunks + vchunks); idx += NWARPS * 32) {
-            const int r = idx / (kchunks + vchunks), c = idx - r * (kchunks + vchunks);
+        // eight lanes a row
+#pragma unroll
+        for (int r0 = 0; r0 < KB; r0 += NWARPS * 4) {
+            const int r = r0 + (threadIdx.x >> 3);
             const int t = min(kb * KB + r, last_pos);                    // rows past the end repeat the last key
-            const int page = mv_read_page(table[t >> page_shift]);
-            const __nv_bfloat16* pbase = pool + (size_t)page * page_stride;
-            const size_t prow = (size_t)g * page_size + (t & (page_size - 1));
-            if (c < kchunks)
-                cp_async16(ks + ((size_t)buf * KB + r) * ldk + c * 8, pbase + prow * dk + c * 8);
-            else
-                cp_async16(vs + ((size_t)buf * KB + r) * ldv + (c - kchunks) * 8,
-                           pbase + v_base + ((size_t)vg * page_size + (t & (page_size - 1))) * v_ld + (c - kchunks) * 8);
+            const __nv_bfloat16* pbase = pool + (size_t)mv_read_page(table[t >> page_shift]) * page_stride;
+            const int in_page = t & (page_size - 1);
+            const __nv_bfloat16* krow = pbase + (size_t)(g * page_size + in_page) * dk;
+            const __nv_bfloat16* vrow = pbase + v_base + (size_t)(vg * page_size + in_page) * v_ld;
+            for (int c = (threadIdx.x & 7) * 8; c < dk; c += 64) cp_async16(ks + (buf * KB + r) * ldk + c, krow + c);
+            for (int c = (threadIdx.x & 7) * 8; c < dv; c += 64) cp_async16(vs + (buf * KB + r) * ldv + c, vrow + c);
         }
     };
     auto block_of = [&](int it) { return it < n_kept ? it : kb_begin + (it - n_kept); };
 
+    const int k_at = ((lane & 7) + ((lane >> 4) & 1) * 8) * ldk + ((lane >> 3) & 1) * 8;      // a lane's row of the keys' fragments
     load_block(block_of(0), 0);
     cp_async_commit();
     for (int it = 0; it < n_iter; ++it) {
@@ -168,16 +188,18 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
         const __nv_bfloat16* vt = vs + (size_t)buf * KB * ldv;
         float s[KB / 8][4];
 #pragma unroll
-        for (int j = 0; j < KB / 8; ++j) {
+        for (int j = 0; j < KB / 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
-            const __nv_bfloat16* krow = kt + (size_t)(j * 8 + gq) * ldk + 2 * t4;
 #pragma unroll
-            for (int kk = 0; kk < DKM / 16; ++kk) {
-                if (kk * 16 < dk) {
-                    const unsigned b0 = *reinterpret_cast<const unsigned*>(krow + kk * 16);
-                    const unsigned b1 = *reinterpret_cast<const unsigned*>(krow + kk * 16 + 8);
-                    mma_bf16(s[j], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b0, b1);
+        for (int kk = 0; kk < DKM / 16; ++kk) {
+            if (kk * 16 < dk) {
+#pragma unroll
+                for (int j = 0; j < KB / 8; j += 2) {
+                    unsigned kf[4];                                      // 16 keys x 16 elements
+                    ldmatrix_x4(kf, kt + k_at + j * 8 * ldk + kk * 16);
+                    mma_bf16(s[j], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], kf[0], kf[1]);
+                    mma_bf16(s[j + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], kf[2], kf[3]);
                 }
             }
         }
@@ -193,21 +215,15 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
         for (int j = 0; j < KB / 8; ++j) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                float sc = s[j][e] * scale;
-                if (cap > 0.f) {
-                    // tanh(x) = (1 - e^-2|x|) / (1 + e^-2|x|) with the fast exponential: within 1e-6 of the capped
-                    // score's size, far below the bfloat16 rounding of the weights that follows
-                    const float x = sc * inv_cap, e2 = __expf(-2.0f * fabsf(x));
-                    sc = copysignf(cap * __fdividef(1.0f - e2, 1.0f + e2), x);
-                }
-                sc += add;
+                float sc = cap > 0.f ? fmaf(-2.0f * cap_l, rcp(1.0f + ex2(s[j][e] * scale_l)), cap_l + add)
+                                     : fmaf(s[j][e], scale_l, add);
                 if (need_mask) {
                     const int t = key0 + j * 8 + 2 * t4 + (e & 1);
                     const int p = (e < 2) ? p0 : p1;
                     if (t > p || (chunk > 0 ? t < ((e < 2) ? cs0 : cs1)
                                             : (window > 0 && t <= p - window && t >= keep_first))) sc = -INFINITY;
                     else if (r1) sc -= db1 * __logf(1.0f + db2 * (float)(p - t));
-                    else if (near) sc += by_dist[min(p - t, dist_len - 1)];
+                    else if (near) sc = fmaf(by_dist[min(p - t, dist_len - 1)], dist_unit, sc);
                 }
                 s[j][e] = sc;
             }
@@ -221,16 +237,16 @@ attention_sink_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bf
         const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
         // a row whose keys are all masked so far (and that has no sink) keeps m = -inf; use 0 as its reference
         const float ref0 = mn0 == -INFINITY ? 0.f : mn0, ref1 = mn1 == -INFINITY ? 0.f : mn1;
-        const float c0 = m0 == -INFINITY ? 0.f : exp2f((m0 - ref0) * LOG2E);
-        const float c1 = m1 == -INFINITY ? 0.f : exp2f((m1 - ref1) * LOG2E);
+        const float c0 = m0 == -INFINITY ? 0.f : ex2(m0 - ref0);
+        const float c1 = m1 == -INFINITY ? 0.f : ex2(m1 - ref1);
         m0 = mn0; m1 = mn1;
         float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
         for (int j = 0; j < KB / 8; ++j) {
-            s[j][0] = exp2f((s[j][0] - ref0) * LOG2E);
-            s[j][1] = exp2f((s[j][1] - ref0) * LOG2E);
-            s[j][2] = exp2f((s[j][2] - ref1) * LOG2E);
-            s[j][3] = exp2f((s[j][3] - ref1) * LOG2E);
+            s[j][0] = ex2(s[j][0] - ref0);
+            s[j][1] = ex2(s[j][1] - ref0);
+            s[j][2] = ex2(s[j][2] - ref1);
+            s[j][3] = ex2(s[j][3] - ref1);
             sum0 += s[j][0] + s[j][1];
             sum1 += s[j][2] + s[j][3];
         }
@@ -317,7 +333,7 @@ int launch(const void* q, const void* pool, long long page_stride, const int* pa
                              (int)((size_t)2 * KB * (DKM + 8 + DVM + 8) * sizeof(__nv_bfloat16) + DIST_SMEM * sizeof(float)));
         attr_set = true;
     }
-    dim3 grid((N + QT - 1) / QT + B, o_all ? nh * nkv : nh);         // an upper bound of the tiles; spare blocks return at once
+    dim3 grid(o_all ? nh * nkv : nh, (N + QT - 1) / QT + B);         // an upper bound of the tiles; spare blocks return at once
     attention_sink_prefill_kernel<DKM, DVM, SPLIT><<<grid, NWARPS * 32, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_stride, page_table, table_stride, page_shift, cu,
         starts, sinks, gate, ld_gate, (__nv_bfloat16*)o, B, nh, nkv, dk, dv, scale, cap, window, keep_first, chunk, r1, r2,
