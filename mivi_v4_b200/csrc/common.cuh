@@ -77,6 +77,13 @@ __device__ __forceinline__ float mv_glu_gelu(float g, float u) {
     const float y2 = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);       // 2 sqrt(2 / pi) (g + 0.044715 g^3)
     return g / (1.0f + expf(-y2)) * u;
 }
+// The same with the hardware's exponential and reciprocal (some 2^-20 off), for results that are rounded to bfloat16 at once.
+// (An exact quotient also takes its slow path where g is zero, as it is wherever an expert was not chosen.)
+__device__ __forceinline__ float mv_glu_silu_fast(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
+__device__ __forceinline__ float mv_glu_gelu_fast(float g, float u) {
+    const float y2 = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
+    return __fdividef(g, 1.0f + __expf(-y2)) * u;
+}
 
 // Loads 8 consecutive elements (16-byte aligned for bf16, 32-byte span for
 // f32) into floats.

@@ -437,7 +437,7 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __
             const float up = __shfl_down_sync(0xffffffffu, v, 16);
             if (lane < 16 && n + 16 < N)
                 ((__nv_bfloat16*)out)[(size_t)m * ldo + (n >> 5) * 16 + lane] =
-                    __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v, up, bias[n], bias[N]) : TAIL == 4 ? mv_glu_gelu(v, up) : mv_glu_silu(v, up));
+                    __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v, up, bias[n], bias[N]) : TAIL == 4 ? mv_glu_gelu_fast(v, up) : mv_glu_silu(v, up));
         } else {
             float sq = 0.f;
             if (r < ROWS && n < N) {

@@ -149,6 +149,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         const int quarter = warp & 3;
         const int row = m0 + quarter * 32 + lane;
         const float ss = row_sum(rs, row, M);            // asked for while the products still run
+        WeightCursor wc;
+        if (ACT == ACT_WEIGHTED) wc.move(rw, row, M, n0 >> 5);
         if (mbar_wait(acc_bar, 0, err, 3)) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const float sc = rs.part ? 1.0f / sqrtf(ss * rs.inv_dim + rs.eps) : 1.f;
@@ -158,7 +160,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 tmem_ld32(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)c0, r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 if (rs.part) scale_chunk(r, sc);
-                if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, rw);
+                if (ACT == ACT_WEIGHTED) wc.move(rw, row, M, (n0 + c0) >> 5);
+                if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, wc.w);
             }
         }
     }
@@ -288,6 +291,8 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             const unsigned acc_phase = (unsigned)(local >> 1) & 1u;
             const int row = m0 + quarter * 32 + lane;
             const float ss = row_sum(rs, row, M);        // asked for while the tile's products still run
+            WeightCursor wc;
+            if (ACT == ACT_WEIGHTED) wc.move(rw, row, M, n0 >> 5);
             ok = mbar_wait(acc_full0 + 8 * acc, acc_phase, err, 3);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -299,7 +304,8 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 tmem_ld32(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)(acc * BN + c0), r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 if (rs.part) scale_chunk(r, sc);
-                if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, rw);
+                if (ACT == ACT_WEIGHTED) wc.move(rw, row, M, (n0 + c0) >> 5);
+                if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, wc.w);
             }
             // this warp has read its lanes of the accumulator: hand it back
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");

@@ -227,6 +227,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 }
             };
             if (link.emit_x) request(0, old);
+            WeightCursor wc;
+            if (ACT == ACT_WEIGHTED) wc.move(rw, row, M, n0 >> 5);
             ok = mbar_wait(acc_full0 + 8 * acc, acc_phase, err, 3);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -305,7 +307,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                         for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
                     }
-                    if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, rw);
+                    if (ACT == ACT_WEIGHTED) wc.move(rw, row, M, (n0 + c0) >> 5);
+                    if (row < M) store_chunk<ACT>(r, row, n0 + c0, N, mode, bias, out, ldo, wc.w);
                 }
             }
             // this warp has read its lanes of the accumulator: tell the leader's MMA warp

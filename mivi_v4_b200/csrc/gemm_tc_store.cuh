@@ -11,13 +11,26 @@ struct RowWeights {
     const float* w;
     int ld, chunks, n_experts;
 };
+// A row's weight for the 32-column chunk c, kept until the next expert's columns begin: a tile mostly holds one expert's,
+// and its weight is asked for before the tile's products are done.
+struct WeightCursor {
+    int end = 0;                   // the chunk where the held weight's expert ends
+    float w = 1.f;
+    __device__ __forceinline__ void move(const RowWeights& rw, int row, int M, int c) {
+        if (c < end) return;
+        const int e = c / rw.chunks;
+        w = e < rw.n_experts && row < M ? rw.w[(size_t)row * rw.ld + e] : 1.f;
+        end = e < rw.n_experts ? (e + 1) * rw.chunks : 0x7fffffff;
+    }
+};
 // One row's 32 consecutive columns of the accumulator, from registers to Y, in the mode asked for.
+// wt: mode 6's weight.
 // ACT: an instance of its own for each of the modes 4, 5 and 6 (the branches would cost the other modes registers).
 enum { ACT_PLAIN = 0, ACT_CLAMPED = 1, ACT_GELU = 2, ACT_WEIGHTED = 3 };
 template <int ACT>
 __device__ __forceinline__ void store_chunk(const unsigned (&r)[32], int row, int n_base, int N, int mode,
                                             const float* __restrict__ bias, void* __restrict__ out, int ldo,
-                                            const RowWeights& rw) {
+                                            float wt) {
 
         constexpr bool CLAMP = ACT == ACT_CLAMPED;
         if (ACT != ACT_PLAIN || mode == 3) {
@@ -26,11 +39,6 @@ __device__ __forceinline__ void store_chunk(const unsigned (&r)[32], int row, in
                 __nv_bfloat16* dst = (__nv_bfloat16*)out + (size_t)row * ldo + (n_base >> 1);
                 unsigned packed[8];
                 const float limit = CLAMP ? bias[n_base] : 0.f, alpha = CLAMP ? bias[N] : 0.f;
-                float wt = 1.f;
-                if (ACT == ACT_WEIGHTED) {
-                    const int e = (n_base >> 5) / rw.chunks;
-                    if (e < rw.n_experts) wt = rw.w[(size_t)row * rw.ld + e];
-                }
 #pragma unroll
                 for (int j = 0; j < 16; j += 2) {
                     float a0 = __uint_as_float(r[j]), a1 = __uint_as_float(r[j + 1]);
@@ -42,7 +50,8 @@ __device__ __forceinline__ void store_chunk(const unsigned (&r)[32], int row, in
                     }
                     const __nv_bfloat162 v =
                         CLAMP ? __floats2bfloat162_rn(mv_glu_clamped(a0, b0, limit, alpha), mv_glu_clamped(a1, b1, limit, alpha))
-                        : ACT == ACT_GELU ? __floats2bfloat162_rn(mv_glu_gelu(a0, b0), mv_glu_gelu(a1, b1))
+                        : ACT == ACT_GELU ? __floats2bfloat162_rn(mv_glu_gelu_fast(a0, b0), mv_glu_gelu_fast(a1, b1))
+                        : ACT == ACT_WEIGHTED ? __floats2bfloat162_rn(mv_glu_silu_fast(a0, b0), mv_glu_silu_fast(a1, b1))
                               : __floats2bfloat162_rn(mv_glu_silu(a0, b0), mv_glu_silu(a1, b1));
                     packed[j >> 1] = *reinterpret_cast<const unsigned*>(&v);
                 }

@@ -388,7 +388,7 @@ gemm_tc_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                         for (int e = 0; e < 4; ++e)
                             o[e] = __float2bfloat16_rn(TAIL == 3 ? mv_glu_clamped(v[e], up[e], bias[n], bias[N])
-                                                      : TAIL == 4 ? mv_glu_gelu(v[e], up[e]) : mv_glu_silu(v[e], up[e]));
+                                                      : TAIL == 4 ? mv_glu_gelu_fast(v[e], up[e]) : mv_glu_silu(v[e], up[e]));
                     }
                 } else {
                     const size_t o = (size_t)m * ldo + n;
