@@ -168,7 +168,7 @@ def _rounded(h, p, dtype):
 
 ATT = [(_m(6, 2, 32, 16, 0.4, 5.0, 0.8, 7, 40), 12, 16), (_m(1, 1, 8, 8, 1.0, 30.0, 0.5, 1, 64), 8, 64),
        (_m(3, 1, 11, 9, 0.5, 2.0, 1.5, 50, 20), 2, 8), (_m(4, 4, 16, 128, 0.7, 8.0, 0.3, 33, 2000), 31, 16),
-       (_m(8, 1, 64, 48, 0.3, 20.0, 0.4, 64, 33), 9, 32), (_m(10, 5, 128, 64, 0.2, 9.0, 0.1, 100, 120), 16, 64),
+       (_m(8, 1, 64, 48, 0.3, 20.0, 0.4, 64, 33), 9, 32), (_m(10, 5, 128, 64, 0.2, 9.0, 0.1, 100, 110), 16, 64),
        (_m(2, 2, 250, 256, 0.2, 4.0, 0.6, 10, 7), 3, 16), (_m(12, 1, 48, 32, 0.4, 6.0, 0.2, 30, 90), 20, 16),
        (_m(40, 2, 16, 16, 0.5, 5.0, 0.4, 25, 50), 6, 8), (_m(5, 5, 256, 256, 0.1, 9.0, 0.3, 12, 30), 10, 16)]
 
